@@ -3,9 +3,11 @@ from .base import (ConfigError, LayerSpec, ModelConfig, ModelSpec, PartSpec, Sch
 from .gatutar import GatutarConfig
 from .kefisun import KefisunConfig
 from .kolorax import KoloraxConfig
+from .mumopel import MumopelConfig
 from .papusun import PapusunConfig
 from .pepolorn import PepolornConfig
 from .qwen3 import Qwen3Config
 
 __all__ = ["ConfigError", "LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "ScheduleEntry",
-           "GatutarConfig", "KefisunConfig", "KoloraxConfig", "PapusunConfig", "PepolornConfig", "Qwen3Config", "read_config_json"]
+           "GatutarConfig", "KefisunConfig", "KoloraxConfig", "MumopelConfig", "PapusunConfig", "PepolornConfig", "Qwen3Config",
+           "read_config_json"]

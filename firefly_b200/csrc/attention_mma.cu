@@ -119,13 +119,16 @@ struct WarpState {
     float o[D / 8][4];
     float m[2], l[2];
 
-    // `sink`: the rows start with one entry of score 0 and no value already taken in (it then stays in the
-    // denominator through every rescale).  The sums of a quad are joined at the end, so one lane of it holds the entry.
-    __device__ __forceinline__ void init(bool sink) {
+    // `s0`, `s1`: the sinks of the thread's two rows, scores without a key and a value that the rows start with (in the
+    // units of the scaled scores, log2 e included; minus infinity: none).  A sink stays in the denominator through every
+    // rescale.  The sums of a quad are joined at the end, so one lane of it holds the entry.
+    __device__ __forceinline__ void init(float s0, float s1) {
 #pragma unroll
         for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
-        m[0] = m[1] = sink ? 0.f : -CUDART_INF_F;
-        l[0] = l[1] = sink && (threadIdx.x & 3) == 0 ? 1.f : 0.f;
+        m[0] = s0;
+        m[1] = s1;
+        l[0] = s0 != -CUDART_INF_F && (threadIdx.x & 3) == 0 ? 1.f : 0.f;
+        l[1] = s1 != -CUDART_INF_F && (threadIdx.x & 3) == 0 ? 1.f : 0.f;
         cap = cap_k = 0.f;
     }
     // a cap on the scores (in the units of the scaled scores, log2 e included; 0: none): v <- cap * tanh(v / cap)
@@ -243,7 +246,7 @@ attn_tiled_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restri
                   const int* __restrict__ block_table, int max_blocks, const int* __restrict__ cu_q,
                   const int* __restrict__ ctx_lens, int n_seqs, bf16* __restrict__ out, int out_stride,
                   int nq, int nkv, int block_size, int num_blocks, float scale_log2, int window,
-                  const float* __restrict__ dist_bias, int bias_len, float softcap_log2, int sink,
+                  const float* __restrict__ dist_bias, int bias_len, float softcap_log2, const float* __restrict__ sink,
                   int* __restrict__ status) {
     pdl_prologue();
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -332,7 +335,12 @@ attn_tiled_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restri
     const int warp_lo = first_visible_key(warp_first_pos, window);   // first key any row sees
 
     WarpState<BN> st;
-    st.init(sink != 0);
+    float s_init[2] = {-CUDART_INF_F, -CUDART_INF_F};
+    if (sink) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) s_init[r] = sink[kh * G + min(row0 + warp * 16 + g + 8 * r, rows - 1) % G] * LOG2E;
+    }
+    st.init(s_init[0], s_init[1]);
     st.set_cap(softcap_log2);
     for (int t = t_begin; t < t_end; ++t) {
         const int buf = (t - t_begin) & 1;
@@ -398,7 +406,7 @@ struct DecodeHeads {
     const float* dist_bias;    // [nq][bias_len] or null: a bias by distance taken off the scores (see WarpState::step)
     int bias_len;
     float softcap_log2;        // a cap on the scaled scores (log2 e included), 0: none
-    int sink;                  // one more entry in every softmax's denominator, of score 0 and without a value
+    const float* sink;         // [nq] or null: one more entry in a head's softmax denominator, of this score, without a value
     float temp_coef;           // heads finished here: q also times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1)
     int temp_every;            // (0: no such factor; it needs q_norm_w)
     int value_is_key;          // heads finished here: the row is q heads | k heads and the raw key is the value
@@ -679,8 +687,15 @@ attn_decode_body(const bf16* __restrict__ q, int q_stride, const bf16* __restric
         }
     }
     WarpState<16> st;
-    if constexpr (HEADS && !XHEADS) st.init(false);
-    else st.init(hd.sink != 0 && split == 0 && warp == 0);        // the entry is taken in once per sequence
+    float s_init[2] = {-CUDART_INF_F, -CUDART_INF_F};
+    if constexpr (!HEADS || XHEADS) {
+        if (hd.sink && split == 0 && warp == 0) {                 // the entry is taken in once per sequence
+#pragma unroll
+            for (int r = 0; r < 2; ++r)
+                if ((lane >> 2) + 8 * r < G) s_init[r] = hd.sink[kh * G + (lane >> 2) + 8 * r] * LOG2E;
+        }
+    }
+    st.init(s_init[0], s_init[1]);
     st.set_cap(hd.softcap_log2);
     for (int t = t_begin; t < t_end; ++t) {
         const int buf = (t - t_begin) & 1;
@@ -774,7 +789,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
                    const int* __restrict__ ctx_lens, bf16* __restrict__ out, int out_stride,
                    float* __restrict__ part_o, float* __restrict__ part_ml, int nq, int nkv,
                    int block_size, int num_blocks, float scale_log2, int window, int num_splits,
-                   const float* __restrict__ dist_bias, int bias_len, float softcap_log2, int sink,
+                   const float* __restrict__ dist_bias, int bias_len, float softcap_log2, const float* __restrict__ sink,
                    int* __restrict__ status) {
     DecodeHeads hd{};
     hd.sink = sink;
@@ -985,7 +1000,7 @@ FF_EXPORT int ff_attn_tiled(const void* q, int q_stride, const void* cache, cons
                             int max_blocks, const int* cu_q, const int* ctx_lens, int n_seqs,
                             int total_tiles, void* out, int out_stride, int nq, int nkv, int block_size,
                             int num_blocks, float scale, int window, const float* dist_bias, int bias_len,
-                            float softcap, int sink, int* status, cudaStream_t stream) {
+                            float softcap, const float* sink, int* status, cudaStream_t stream) {
     if (n_seqs <= 0 || total_tiles <= 0) return 0;
     if (nkv <= 0 || nq % nkv || (dist_bias && (window <= 0 || bias_len < window))) return FF_ERR_BAD_ARG;
     FF_SMEM_LIMIT(attn_tiled_kernel, TILED_SMEM);
@@ -1004,7 +1019,7 @@ FF_EXPORT int ff_attn_decode(const void* q, int q_stride, const void* cache, con
                              int max_blocks, const int* cu_q, const int* ctx_lens, int n_seqs, void* out,
                              int out_stride, float* part_o, float* part_ml, int nq, int nkv,
                              int block_size, int num_blocks, float scale, int window, int num_splits,
-                             const float* dist_bias, int bias_len, float softcap, int sink, int* status,
+                             const float* dist_bias, int bias_len, float softcap, const float* sink, int* status,
                              cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (nkv <= 0 || nq % nkv || num_splits < 1 || (dist_bias && (window <= 0 || bias_len < window))) return FF_ERR_BAD_ARG;
@@ -1039,7 +1054,7 @@ FF_EXPORT int ff_attn_decode_heads(const void* qkv, int row_width, void* cache, 
                                    int out_stride, float* part_o, float* part_ml, int nq, int nkv,
                                    int block_size, int num_blocks, float scale, int window, int num_splits,
                                    const float* q_norm_w, const float* k_norm_w, float eps,
-                                   const float* cos_sin, int max_positions, int sink, float temp_coef, int temp_every,
+                                   const float* cos_sin, int max_positions, const float* sink, float temp_coef, int temp_every,
                                    int value_is_key, int* status, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (nkv <= 0 || nq % nkv || num_splits < 1 || status == nullptr) return FF_ERR_BAD_ARG;
@@ -1084,7 +1099,7 @@ FF_EXPORT int ff_attn_decode_units(const void* q, int q_stride, void* cache, con
                                    int nkv, int block_size, int num_blocks, float scale, int window, int units,
                                    int max_ranges, int finish_heads, const float* q_norm_w,
                                    const float* k_norm_w, float eps, const float* cos_sin, int max_positions,
-                                   const float* dist_bias, int bias_len, float softcap, int sink, float temp_coef,
+                                   const float* dist_bias, int bias_len, float softcap, const float* sink, float temp_coef,
                                    int temp_every, int value_is_key, int* status, cudaStream_t stream) {
     if (finish_heads && temp_every > 0 && !q_norm_w) return FF_ERR_BAD_ARG;
     if (FF_KV_PLANES != 2 && finish_heads) return FF_ERR_UNSUPPORTED;

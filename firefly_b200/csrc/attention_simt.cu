@@ -38,7 +38,7 @@ __global__ void paged_attention_simt_kernel(
     const int* __restrict__ block_table, int max_blocks, const int* __restrict__ token_seq,
     const int* __restrict__ positions, T* __restrict__ out, int out_stride, int nq, int nkv, int d,
     int block_size, int num_blocks, float scale, int window, const float* __restrict__ dist_bias, int bias_len,
-    float softcap, int sink, int* __restrict__ status) {
+    float softcap, const float* __restrict__ sink, int* __restrict__ status) {
     pdl_prologue();
     q = pdl_fresh(q);              // the kernel in front writes the finished heads and this step's cache rows
     cache = pdl_fresh(cache);
@@ -61,8 +61,8 @@ __global__ void paged_attention_simt_kernel(
         qr[jj] = i < d ? to_float(qrow[i]) : 0.f;
         acc[jj] = 0.f;
     }
-    // a sink (one more entry in the denominator, of score 0 and without a value) is taken in by the first warp
-    float m = sink && warp == 0 ? 0.f : -CUDART_INF_F, l = sink && warp == 0 ? 1.f : 0.f;
+    // a sink (one more entry in the head's denominator, of this score and without a value) is taken in by the first warp
+    float m = sink && warp == 0 ? sink[h] : -CUDART_INF_F, l = sink && warp == 0 ? 1.f : 0.f;
     const int* bt = block_table + (size_t)seq * max_blocks;
     for (int j = kv_begin + warp; j < kv_end; j += ATT_WARPS) {
         const int page = bt[j / block_size];
@@ -125,7 +125,7 @@ FF_EXPORT int ff_paged_attention_simt(const void* q, int dtype, int q_stride, co
                                       const int* block_table, int max_blocks, const int* token_seq,
                                       const int* positions, void* out, int out_stride, int T, int nq,
                                       int nkv, int d, int block_size, int num_blocks, float scale,
-                                      int window, const float* dist_bias, int bias_len, float softcap, int sink, int* status,
+                                      int window, const float* dist_bias, int bias_len, float softcap, const float* sink, int* status,
                                       cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0 || d > ATT_MAX_D) return FF_ERR_UNSUPPORTED;

@@ -216,10 +216,11 @@ attn_tc_kernel(const __grid_constant__ TensorMapArg kv_map, const bf16* __restri
                const int* __restrict__ ctx_lens, int n_seqs, bf16* __restrict__ out, int out_stride, int nq,
                int nkv, int block_size, int num_blocks, float scale_log2, int window, int* __restrict__ status,
                int num_splits, float* __restrict__ part_o, float* __restrict__ part_ml,
-               const float* __restrict__ dist_bias, int bias_len, float softcap_log2, int sink) {
+               const float* __restrict__ dist_bias, int bias_len, float softcap_log2, const float* __restrict__ sink) {
     // dist_bias (float [nq][bias_len >= window], or null): entry (head, i - j) is taken off the scaled score of
     // query position i and key position j; a window lets only distances below `window` through.
-    // sink: one more entry in every softmax's denominator, of score 0 and without a value; the first share takes it in.
+    // sink (float [nq], or null): one more entry in a head's softmax denominator, of this score and without a value; the
+    // first share takes it in.
     // num_splits > 1: the grid holds every (row tile, kv head) num_splits times; each copy walks its share
     // of the tile's keys and leaves an unnormalised result with its (reference max, sum) for the join
     // kernel.  For prompts so short that their row tiles would leave most SMs idle while each block
@@ -375,8 +376,8 @@ attn_tc_kernel(const __grid_constant__ TensorMapArg kv_map, const bf16* __restri
         const bool early = dist_bias != nullptr || softcap_log2 != 0.f;
         const float sl2 = early ? 1.0f : scale_log2;
         const float cap_k = softcap_log2 != 0.f ? 2.0f * LOG2E / softcap_log2 : 0.f;
-        const bool has_sink = sink != 0 && split == 0;
-        float m = has_sink ? 0.f : -CUDART_INF_F, l = has_sink ? 1.f : 0.f;
+        const bool has_sink = sink != nullptr && split == 0;
+        float m = has_sink ? sink[head] * LOG2E : -CUDART_INF_F, l = has_sink ? 1.f : 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; ++j) {
             ok = mb_wait(sa(&bars[B_S_FULL + (j & 1)]), (j >> 1) & 1, status, abort_flag);
@@ -710,7 +711,7 @@ FF_EXPORT int ff_attn_tc(const void* q, int q_stride, const void* cache, const i
                          const int* cu_q, const int* ctx_lens, int n_seqs, int total_tiles, void* out,
                          int out_stride, int nq, int nkv, int block_size, int num_blocks, float scale, int window,
                          int* status, int num_splits, float* part_o, float* part_ml, int tok_base, int n_tokens,
-                         const float* dist_bias, int bias_len, float softcap, int sink, cudaStream_t stream) {
+                         const float* dist_bias, int bias_len, float softcap, const float* sink, cudaStream_t stream) {
     if (n_seqs <= 0 || total_tiles <= 0) return 0;
     if (nkv <= 0 || nq % nkv || (dist_bias && (window <= 0 || bias_len < window))) return FF_ERR_BAD_ARG;
     if (num_splits < 1 || (num_splits > 1 && (!part_o || !part_ml || n_tokens <= 0 || tok_base < 0))) return FF_ERR_BAD_ARG;

@@ -506,6 +506,14 @@ __global__ void scale_kernel(float* x, float a, size_t total) {
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx < total) x[idx] *= a;
 }
+
+// x = cap * tanh(x / cap)
+__global__ void softcap_kernel(float* x, float cap, size_t total) {
+    pdl_prologue();
+    x = pdl_fresh(x);
+    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx < total) x[idx] = cap * tanhf(x[idx] / cap);
+}
 }  // namespace ff
 
 FF_EXPORT int ff_norm_add(float* residual, const void* delta, int delta_dtype, const float* w, float eps, void* copy,
@@ -560,6 +568,14 @@ FF_EXPORT int ff_glu_act(const void* gate_up, const float* bias, void* out, int 
     if (dtype == 0) FF_LAUNCH((glu_act_kernel<float>), blocks, 256, 0, stream, (const float*)gate_up, bias, (float*)out, I, total, act, limit);
     else if (dtype == 1) FF_LAUNCH((glu_act_kernel<bf16>), blocks, 256, 0, stream, (const bf16*)gate_up, bias, (bf16*)out, I, total, act, limit);
     else return FF_ERR_BAD_ARG;
+    FF_LAUNCH_CHECK();
+    return 0;
+}
+
+FF_EXPORT int ff_softcap(float* x, float cap, size_t n, cudaStream_t stream) {
+    if (n == 0) return 0;
+    if (!(cap > 0.f)) return FF_ERR_BAD_ARG;
+    FF_LAUNCH(softcap_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, x, cap, n);
     FF_LAUNCH_CHECK();
     return 0;
 }

@@ -2,7 +2,9 @@
 //
 // In the order in which they are applied, each of them optional:
 //   `bias`         (float [(nq + 2 nkv) d] in the row's layout) added to q, k and v in 32-bit;
-//   `q_w`, `k_w`   (float [d]) an RMS norm of every q / k head over its `norm_dim` elements with this weight;
+//   `q_w`, `k_w`   (float [d]) an RMS norm of every q / k head over its `norm_dim` elements with this weight; with
+//                  `norm_all` (float [nq d] / [nkv d]) one norm over all q heads together and one over all k heads, each head
+//                  counting `norm_dim` elements;
 //   rotation       of the first `rdims` elements of every q and k head (pairs (i, i + rdims/2), or (2i, 2i + 1) with
 //                  `interleaved`; angle = position * f_i, cos and sin times `mag`);
 //   `normalize`    q and k divided by their root mean square over `norm_dim` elements (no weight);
@@ -37,6 +39,7 @@ struct HeadFinish {
     int temp_every;
     int value_is_key;
     int T;
+    int norm_all;
 };
 
 // Any type and size: one block a token, one warp a head.
@@ -73,6 +76,19 @@ __global__ void head_finish_kernel(T* __restrict__ qkv, T* __restrict__ cache /*
     }
     const float temp = A.temp_every > 0 ? query_temperature(pos, A.temp_coef, A.temp_every) : 1.0f;
     const int heads = nq + (A.value_is_key ? nkv : 2 * nkv);
+    float inv_q = 1.f, inv_k = 1.f;          // norm_all: 1 / root mean square of all q heads, of all k heads
+    if (A.norm_all) {
+        __shared__ float scratch[32];
+        float sq = 0.f, sk = 0.f;
+        for (int i = threadIdx.x; i < (nq + nkv) * d; i += blockDim.x) {
+            const float v = to_float(row[i]) + (A.bias ? A.bias[i] : 0.f);
+            if (i < nq * d) sq += v * v;
+            else sk += v * v;
+        }
+        inv_q = 1.0f / sqrtf(block_sum(sq, scratch) / (float)(nq * A.norm_dim) + A.eps);
+        if (nkv > 0) inv_k = 1.0f / sqrtf(block_sum(sk, scratch) / (float)(nkv * A.norm_dim) + A.eps);
+        __syncthreads();                     // q is rewritten in place below
+    }
     for (int h = warp; h < heads; h += nwarps) {
         T* src = row + (size_t)h * d;
         const float* brow = A.bias ? A.bias + (size_t)h * d : nullptr;
@@ -95,7 +111,8 @@ __global__ void head_finish_kernel(T* __restrict__ qkv, T* __restrict__ cache /*
             ss += v * v;
         }
         if (w) {
-            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)A.norm_dim + A.eps);
+            const float inv = A.norm_all ? (is_k ? inv_k : inv_q) : 1.0f / sqrtf(warp_sum(ss) / (float)A.norm_dim + A.eps);
+            if (A.norm_all) w += (size_t)(is_k ? h - nq : h) * d;
             for (int i = lane; i < d; i += 32) hbuf[i] = hbuf[i] * inv * w[i];
         }
         __syncwarp();
@@ -130,11 +147,12 @@ __global__ void head_finish_kernel(T* __restrict__ qkv, T* __restrict__ cache /*
 // angles in shared memory) and its warps the heads of all of them, HFV_U passes with their loads in flight together.
 constexpr int HFV_TOK = 4, HFV_THREADS = 256, HFV_U = 4;
 
-template <int P>
+template <int P, bool ALL>
 __global__ void __launch_bounds__(HFV_THREADS) head_finish_vec_kernel(bf16* __restrict__ qkv, bf16* __restrict__ cache, HeadFinish A) {
     extern __shared__ float sh[];                             // [HFV_TOK][2][half]
     __shared__ int s_page[HFV_TOK];
     __shared__ float s_temp[HFV_TOK];
+    __shared__ float s_part[HFV_TOK][2][2], s_inv[HFV_TOK][2];
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int t0 = blockIdx.x * HFV_TOK, nt = min(HFV_TOK, A.T - t0);
     const int d = A.d, nq = A.nq, nkv = A.nkv, half = A.rdims / 2;
@@ -166,6 +184,39 @@ __global__ void __launch_bounds__(HFV_THREADS) head_finish_vec_kernel(bf16* __re
     const int items = nt * heads;                             // (token, head) pairs of the block
     const int passes = (items + HPW - 1) / HPW;
     const bool turns = e0 < A.rdims;
+    if constexpr (ALL) {
+        // sums over all q heads and over all k heads: two warps a token, each every other group of 32 x 8 elements; the
+        // rows are read again below (from the cache then)
+        static_assert(HFV_TOK * 2 == HFV_THREADS / 32, "two warps a token");
+        const int tl = warp >> 1, part = warp & 1;
+        float s[2] = {0.f, 0.f};
+        if (tl < nt) {
+            const bf16* row = qkv + (size_t)(t0 + tl) * A.width;
+            const int nq8 = nq * d / 8, all8 = (nq + nkv) * d / 8;
+#pragma unroll 4
+            for (int c = part * 32 + lane; c < all8; c += 64) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(row + (size_t)c * 8);
+                const bf16* rb = reinterpret_cast<const bf16*>(&raw);
+                float ss = 0.f;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const float v = __bfloat162float(rb[j]) + (A.bias ? A.bias[c * 8 + j] : 0.f);
+                    ss += v * v;
+                }
+                if (c < nq8) s[0] += ss;
+                else s[1] += ss;
+            }
+        }
+        s[0] = warp_sum(s[0]);
+        s[1] = warp_sum(s[1]);
+        if (lane == 0) { s_part[tl][part][0] = s[0]; s_part[tl][part][1] = s[1]; }
+        __syncthreads();
+        if ((int)threadIdx.x < HFV_TOK * 2) {
+            const int u = threadIdx.x >> 1, kind = threadIdx.x & 1, n = (kind ? nkv : nq) * A.norm_dim;
+            s_inv[u][kind] = 1.0f / sqrtf((s_part[u][0][kind] + s_part[u][1][kind]) / (float)max(n, 1) + A.eps);
+        }
+        __syncthreads();
+    }
     const int hl = half / 8;                                  // lanes a half of the rotated elements takes
     const bool upper = turns && !A.interleaved && e0 >= half;
     for (int p0 = warp; p0 < passes; p0 += nwarps * HFV_U) {
@@ -207,7 +258,15 @@ __global__ void __launch_bounds__(HFV_THREADS) head_finish_vec_kernel(bf16* __re
                 put(krow + (size_t)(nkv + h - nq - (is_v ? nkv : 0)) * A.block_size * d);
             // values stay in the shuffles below with the rest of their warp
             const float* w = is_v ? nullptr : (is_k ? A.k_w : A.q_w);
-            if (A.q_w || A.k_w) {
+            if constexpr (ALL) {
+                if (w && live) {
+                    const float inv = s_inv[tl][is_k ? 1 : 0];
+                    const float4* wh = reinterpret_cast<const float4*>(w + (size_t)(is_k ? h - nq : h) * d + e0);
+                    const float4 w0 = wh[0], w1 = wh[1];
+                    v[0] *= inv * w0.x; v[1] *= inv * w0.y; v[2] *= inv * w0.z; v[3] *= inv * w0.w;
+                    v[4] *= inv * w1.x; v[5] *= inv * w1.y; v[6] *= inv * w1.z; v[7] *= inv * w1.w;
+                }
+            } else if (A.q_w || A.k_w) {
                 float ss = 0.f;
 #pragma unroll
                 for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
@@ -268,18 +327,23 @@ FF_EXPORT int ff_head_finish(void* qkv, int dtype, int width, int T, int nq, int
                              const double* freq, int rdims, float mag, const int* positions, const int* token_seq,
                              const int* block_table, int max_blocks, int block_size, int num_blocks, void* cache,
                              int* status, int interleaved, int normalize, const float* bias, const float* q_w,
-                             const float* k_w, float temp_coef, int temp_every, int value_is_key, cudaStream_t stream) {
+                             const float* k_w, float temp_coef, int temp_every, int value_is_key, int norm_all, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (rdims < 0 || rdims % 2 || rdims > d || norm_dim <= 0 || norm_dim > d || d > 1024) return FF_ERR_BAD_ARG;
     const int heads = nq + (value_is_key ? nkv : 2 * nkv);
-    if (width < heads * d) return FF_ERR_BAD_ARG;
+    if (width < heads * d || (norm_all && (!q_w || (nkv > 0 && !k_w)))) return FF_ERR_BAD_ARG;
     HeadFinish A{width, nq, nkv, d, norm_dim, eps, freq, rdims, mag, positions, token_seq, block_table, max_blocks, block_size,
-                 num_blocks, status, interleaved, normalize, bias, q_w, k_w, temp_coef, temp_every, value_is_key, T};
+                 num_blocks, status, interleaved, normalize, bias, q_w, k_w, temp_coef, temp_every, value_is_key, T, norm_all};
     const bool pairs_fit = rdims % 8 == 0 && (interleaved || (rdims / 2) % 8 == 0);
-    if (dtype == 1 && d % 8 == 0 && d <= 256 && width % 8 == 0 && pairs_fit && (((uintptr_t)qkv | (uintptr_t)cache) & 15) == 0) {
+    if (dtype == 1 && d % 8 == 0 && d <= 256 && width % 8 == 0 && pairs_fit && (((uintptr_t)qkv | (uintptr_t)cache) & 15) == 0 &&
+        (!norm_all || (((uintptr_t)q_w | (uintptr_t)k_w) & 15) == 0)) {
         const size_t smem = (size_t)HFV_TOK * rdims * sizeof(float);
         const unsigned blocks = (unsigned)((T + HFV_TOK - 1) / HFV_TOK);
-#define FF_HFV(P) FF_LAUNCH((head_finish_vec_kernel<P>), blocks, HFV_THREADS, smem, stream, (bf16*)qkv, (bf16*)cache, A)
+#define FF_HFV(P)                                                                                                       \
+    do {                                                                                                                \
+        if (norm_all) FF_LAUNCH((head_finish_vec_kernel<P, true>), blocks, HFV_THREADS, smem, stream, (bf16*)qkv, (bf16*)cache, A); \
+        else FF_LAUNCH((head_finish_vec_kernel<P, false>), blocks, HFV_THREADS, smem, stream, (bf16*)qkv, (bf16*)cache, A); \
+    } while (0)
         if (d <= 32) FF_HFV(4);
         else if (d <= 64) FF_HFV(8);
         else if (d <= 128) FF_HFV(16);

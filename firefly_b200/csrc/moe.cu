@@ -40,12 +40,13 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
     }
 }
 
-// One warp per token.  score 0: s = softmax(z) over all experts; 1: s = sigmoid(z).  The choice uses
+// One warp per token; z + bias (bias may be null) are the logits.  score 0: s = softmax(z) over all experts; 1: s =
+// sigmoid(z); 2: s = z, and the weights are the softmax over the chosen experts' logits alone.  The choice uses
 // c = s + correction (correction may be null); a group's score is its largest c (group_score 0) or the sum of
 // its two largest (1); experts of closed groups count as minus infinity (c may be negative); the weights are the
 // chosen experts' s, divided by their sum (+ 1e-20) when `renorm`.  Ties go to the lowest index.
 // z rows are z_stride floats apart (further columns may follow the experts' logits).
-__global__ void moe_route_kernel(const float* z, int z_stride, const float* __restrict__ correction, int T, int E, int top,
+__global__ void moe_route_kernel(const float* z, int z_stride, const float* __restrict__ bias, const float* __restrict__ correction, int T, int E, int top,
                                  int groups, int keep, int score, int group_score, int renorm,
                                  int* __restrict__ ids, float* __restrict__ wts) {
     pdl_prologue();
@@ -59,17 +60,20 @@ __global__ void moe_route_kernel(const float* z, int z_stride, const float* __re
     float* gs = a + E;
     float* g_open = gs + groups;
     const float* zr = z + (size_t)t * z_stride;
+    float mx = -CUDART_INF_F;
+    for (int e = lane; e < E; e += 32) {
+        s[e] = zr[e] + (bias ? bias[e] : 0.f);
+        mx = fmaxf(mx, s[e]);
+    }
     if (score == 0) {
-        float mx = -CUDART_INF_F;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e]);
         mx = warp_max(mx);
         float sum = 0.f;
-        for (int e = lane; e < E; e += 32) { const float p = expf(zr[e] - mx); s[e] = p; sum += p; }
+        for (int e = lane; e < E; e += 32) { const float p = expf(s[e] - mx); s[e] = p; sum += p; }
         sum = warp_sum(sum);
         __syncwarp();
         for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
-    } else {
-        for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-zr[e]));
+    } else if (score == 1) {
+        for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
     }
     __syncwarp();
     const int per = E / groups;
@@ -95,7 +99,7 @@ __global__ void moe_route_kernel(const float* z, int z_stride, const float* __re
     for (int e = lane; e < E; e += 32)
         a[e] = g_open[e / per] != 0.f ? s[e] + (correction ? correction[e] : 0.f) : -CUDART_INF_F;
     __syncwarp();
-    float total = 0.f;
+    float total = 0.f, largest = -CUDART_INF_F;
     for (int k = 0; k < top; ++k) {
         float bv = -CUDART_INF_F;
         int bi = 0x7fffffff;
@@ -105,10 +109,16 @@ __global__ void moe_route_kernel(const float* z, int z_stride, const float* __re
         if (bi >= E) bi = 0;                   // cannot happen: top <= keep * per open experts with finite scores
         const float w = s[bi];
         total += w;
+        largest = fmaxf(largest, w);
         if (lane == 0) { ids[(size_t)t * top + k] = bi; wts[(size_t)t * top + k] = w; a[bi] = -CUDART_INF_F; }
         __syncwarp();
     }
-    if (renorm) {
+    if (score == 2) {
+        total = 0.f;
+        for (int k = lane; k < top; k += 32) total += expf(wts[(size_t)t * top + k] - largest);
+        total = warp_sum(total);
+        for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] = expf(wts[(size_t)t * top + k] - largest) / total;
+    } else if (renorm) {
         const float inv = 1.0f / (total + 1e-20f);
         __syncwarp();
         for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] *= inv;
@@ -417,7 +427,7 @@ using namespace ff;
 // rows of a row tile: of the tensor-core kernel (bfloat16, K % 8 == 0) or of the plain one
 FF_EXPORT int ff_moe_row_tile(int tensor_cores) { return tensor_cores ? MMA_BM : MOE_BM; }
 
-FF_EXPORT int ff_moe_route(const float* z, int z_stride, const float* correction, int T, int E, int top, int groups, int keep,
+FF_EXPORT int ff_moe_route(const float* z, int z_stride, const float* bias, const float* correction, int T, int E, int top, int groups, int keep,
                            int score, int group_score, int renorm, int* ids, float* wts, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (E <= 0 || z_stride < E || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
@@ -426,7 +436,7 @@ FF_EXPORT int ff_moe_route(const float* z, int z_stride, const float* correction
     const int warps = 4;
     const size_t smem = (size_t)warps * (2 * E + 2 * groups) * sizeof(float);
     if (smem > 48 * 1024) return FF_ERR_UNSUPPORTED;
-    FF_LAUNCH(moe_route_kernel, (T + warps - 1) / warps, warps * 32, smem, stream, z, z_stride, correction, T, E, top, groups, keep, score,
+    FF_LAUNCH(moe_route_kernel, (T + warps - 1) / warps, warps * 32, smem, stream, z, z_stride, bias, correction, T, E, top, groups, keep, score,
               group_score, renorm, ids, wts);
     FF_LAUNCH_CHECK();
     return 0;

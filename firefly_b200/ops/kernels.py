@@ -10,7 +10,7 @@ from __future__ import annotations
 import ctypes
 import functools
 from ctypes import c_float, c_int, c_size_t, c_void_p
-from typing import Optional
+from typing import Optional, Union
 
 import torch
 
@@ -87,6 +87,7 @@ _MODULES = {
     "conv_attention": ("conv_attention.cu", None),
     "delta_rule": ("delta_rule.cu", None),
     "sandwich_norm": ("sandwich_norm.cu", None),
+    "stream_seam": ("stream_seam.cu", None),
 }
 
 
@@ -231,17 +232,42 @@ def _check_dist_bias(dist_bias: Optional[torch.Tensor], nq: int, window: int) ->
         raise KernelError("attention: a bias by distance needs a window no longer than its table")
 
 
+Sink = Union[None, bool, torch.Tensor]
+_ZERO_SINKS = {}
+
+
+def _zero_sinks(device: torch.device) -> torch.Tensor:
+    """Scores of 0 for up to 1024 heads, made once per device."""
+    z = _ZERO_SINKS.get(device)
+    if z is None:
+        if torch.cuda.is_current_stream_capturing():
+            raise KernelError("attention: run a step with sinks once before the capture")
+        z = _ZERO_SINKS[device] = torch.zeros(1024, dtype=torch.float32, device=device)
+        torch.cuda.synchronize(device)          # kernels may read it in front of their wait for the stream
+    return z
+
+
+def _sink_arg(sink: Sink, nq: int) -> c_void_p:
+    if sink is None or sink is False:
+        return c_void_p(0)
+    if sink is True:
+        sink = _zero_sinks(torch.device("cuda", torch.cuda.current_device()))
+    if not sink.is_cuda or sink.dtype != torch.float32 or sink.numel() < nq or not sink.is_contiguous():
+        raise KernelError("attention: the sinks are a contiguous float32 tensor, one score a query head")
+    return _p(sink)
+
+
 def paged_attention_simt(q: torch.Tensor, q_stride: int, cache: torch.Tensor, block_table: torch.Tensor,
                          token_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor,
                          nq: int, nkv: int, d: int, scale: float, window: int,
                          status: torch.Tensor, dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                         sink: bool = False) -> None:
+                         sink: Sink = None) -> None:
     """Attention of every query token over its sequence's cached keys 0..pos
     (or the last ``window`` of them; 0 = all).  ``q`` is read with row stride
     ``q_stride`` elements (it may be the head of a wider qkv buffer).  ``dist_bias`` float32 [nq, L]:
     entry (h, i - j) is taken off the score of query position i and key position j.  ``softcap`` c > 0: the scaled score
-    s becomes c tanh(s / c) (before the bias).  ``sink``: one more entry in the softmax's denominator, of score 0 and
-    without a value."""
+    s becomes c tanh(s / c) (before the bias).  ``sink`` float32 [nq]: one more entry in every softmax's denominator, of the
+    head's score as given (not scaled, not capped) and without a value; True: of score 0 for every head."""
     _need_cuda(cache, block_table, token_seq, positions, out, status, dist_bias)
     _check_dist_bias(dist_bias, nq, window)
     if not q.is_cuda:
@@ -254,7 +280,7 @@ def paged_attention_simt(q: torch.Tensor, q_stride: int, cache: torch.Tensor, bl
         _p(q), c_int(_dt(q)), c_int(q_stride), _p(cache), _p(block_table), c_int(block_table.shape[1]),
         _p(token_seq), _p(positions), _p(out), c_int(out.shape[1]), c_int(T), c_int(nq), c_int(nkv),
         c_int(d), c_int(block_size), c_int(num_blocks), c_float(scale), c_int(window), _p(dist_bias),
-        c_int(dist_bias.shape[1] if dist_bias is not None else 0), c_float(softcap), c_int(1 if sink else 0), _p(status),
+        c_int(dist_bias.shape[1] if dist_bias is not None else 0), c_float(softcap), _sink_arg(sink, nq), _p(status),
         _stream()), "paged_attention_simt")
 
 
@@ -493,7 +519,7 @@ def _bias_args(dist_bias: Optional[torch.Tensor], nq: int, window: int):
 
 def attn_tiled(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, total_tiles, out, nq, nkv, d, scale,
                window, status: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
-               softcap: float = 0.0, sink: bool = False) -> None:
+               softcap: float = 0.0, sink: Sink = None) -> None:
     """Tensor-core attention for any mix of sequences (bfloat16).  ``status`` (int32 [1]) is set to 4
     when a key that must be read has no valid page in the block table.  ``dist_bias``, ``sink``: as for
     `paged_attention_simt`."""
@@ -503,12 +529,12 @@ def attn_tiled(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, total_tiles, o
         _p(q), c_int(q_stride), _p(pages), _p(table), c_int(table.shape[1]), _p(cu_q), _p(ctx_lens),
         c_int(n_seqs), c_int(total_tiles), _p(out), c_int(out.shape[1]), c_int(nq), c_int(nkv),
         c_int(block_size), c_int(num_blocks), c_float(scale), c_int(window), *_bias_args(dist_bias, nq, window),
-        c_float(softcap), c_int(1 if sink else 0), _p(status), _stream()), "attn_tiled")
+        c_float(softcap), _sink_arg(sink, nq), _p(status), _stream()), "attn_tiled")
 
 
 def attn_decode(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, out, part_o, part_ml, nq, nkv, d,
                 scale, window, num_splits, status: Optional[torch.Tensor] = None,
-                dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0, sink: bool = False) -> None:
+                dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0, sink: Sink = None) -> None:
     """Split-KV tensor-core attention when every sequence has one token (bfloat16).  ``status``,
     ``dist_bias`` and ``sink`` as for `attn_tiled`."""
     _need_cuda(pages, table, cu_q, ctx_lens, out, part_o, part_ml, status, dist_bias)
@@ -517,7 +543,7 @@ def attn_decode(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, out, part_o, 
         _p(q), c_int(q_stride), _p(pages), _p(table), c_int(table.shape[1]), _p(cu_q), _p(ctx_lens),
         c_int(n_seqs), _p(out), c_int(out.shape[1]), _p(part_o), _p(part_ml), c_int(nq), c_int(nkv),
         c_int(block_size), c_int(num_blocks), c_float(scale), c_int(window), c_int(num_splits),
-        *_bias_args(dist_bias, nq, window), c_float(softcap), c_int(1 if sink else 0), _p(status), _stream()), "attn_decode")
+        *_bias_args(dist_bias, nq, window), c_float(softcap), _sink_arg(sink, nq), _p(status), _stream()), "attn_decode")
     global LAUNCHES
     if num_splits > 1:
         LAUNCHES += 1     # the kernel that joins the splits
@@ -541,7 +567,7 @@ def decode_finishes_heads(ctx, dtype: torch.dtype, nq: int, nkv: int, d: int, ro
 
 
 def attn_decode_heads(qkv, pages, table, ctx, out, nq, nkv, d, scale, window, q_norm_w, k_norm_w, eps,
-                      cos_sin, num_splits: Optional[int] = None, *, sink: bool = False, q_temp=None,
+                      cos_sin, num_splits: Optional[int] = None, *, sink: Sink = None, q_temp=None,
                       value_is_key: bool = False) -> None:
     """The split-KV decode attention fed with the raw q|k|v projection ``[T, (nq + 2 nkv) d]``:
     it finishes the heads itself (per-head RMSNorm, rotation, cache write of the newest key and
@@ -568,7 +594,7 @@ def attn_decode_heads(qkv, pages, table, ctx, out, nq, nkv, d, scale, window, q_
         c_int(n), _p(out), c_int(out.shape[1]), _p(part_o), _p(part_ml), c_int(nq), c_int(nkv),
         c_int(block_size), c_int(num_blocks), c_float(scale), c_int(window), c_int(splits),
         _p(q_norm_w), _p(k_norm_w), c_float(eps), _p(cos_sin), c_int(cos_sin.shape[0] if cos_sin is not None else 0),
-        c_int(1 if sink else 0), *_temp_args(q_temp), c_int(1 if value_is_key else 0), _p(ctx.status), _stream()),
+        _sink_arg(sink, nq), *_temp_args(q_temp), c_int(1 if value_is_key else 0), _p(ctx.status), _stream()),
         "attn_decode_heads")
     if splits > 1:
         LAUNCHES += 1     # the kernel that joins the splits
@@ -592,7 +618,7 @@ def tc_attention_supported(dtype: torch.dtype, d: int, block_size: int, max_kv_l
 
 def attn_tc(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, total_tiles, out, nq, nkv, d, scale, window,
             status, page_list: Optional[int] = None, shares=None, dist_bias: Optional[torch.Tensor] = None,
-            softcap: float = 0.0, sink: bool = False) -> None:
+            softcap: float = 0.0, sink: Sink = None) -> None:
     """tcgen05 flash attention over the paged cache (bfloat16); total_tiles counts row tiles of 128.
     ``shares`` = (count, part_o, part_ml, first row, rows): every row tile's keys are shared out over
     ``count`` blocks and a second kernel joins their partial results (for prompts so short that their
@@ -610,7 +636,7 @@ def attn_tc(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, total_tiles, out,
         c_int(n_seqs), c_int(total_tiles), _p(out), c_int(out.shape[1]), c_int(nq), c_int(nkv),
         c_int(block_size), c_int(num_blocks), c_float(scale), c_int(window), _p(status), c_int(count), _p(part_o),
         _p(part_ml), c_int(row0), c_int(rows), *_bias_args(dist_bias, nq, window), c_float(softcap),
-        c_int(1 if sink else 0), _stream()), "attn_tc")
+        _sink_arg(sink, nq), _stream()), "attn_tc")
     if count > 1:
         global LAUNCHES
         LAUNCHES += 1     # the kernel that joins the shares
@@ -693,7 +719,7 @@ def _decode_scratch(ws, n: int, nq: int, nkv: int, d: int, splits: int):
 
 def attn_decode_units(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, out, part_o, part_ml, seq_ranges,
                       nq, nkv, d, scale, window, units, max_ranges, heads=None, status=None,
-                      dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0, sink: bool = False, q_temp=None,
+                      dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0, sink: Sink = None, q_temp=None,
                       value_is_key: bool = False) -> None:
     """Split-KV decode attention with `units` blocks per kv head shared out among the sequences
     in proportion to their lengths.  ``heads = (q_norm_w, k_norm_w, eps, cos_sin)``: q is the raw
@@ -710,7 +736,7 @@ def attn_decode_units(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, out, pa
         c_int(nkv), c_int(block_size), c_int(num_blocks), c_float(scale), c_int(window), c_int(units),
         c_int(max_ranges), c_int(1 if heads is not None else 0), _p(qw), _p(kw), c_float(eps), _p(cos_sin),
         c_int(cos_sin.shape[0] if cos_sin is not None else 0), *_bias_args(dist_bias, nq, window), c_float(softcap),
-        c_int(1 if sink else 0), *_temp_args(q_temp), c_int(1 if value_is_key else 0), _p(status), _stream()),
+        _sink_arg(sink, nq), *_temp_args(q_temp), c_int(1 if value_is_key else 0), _p(status), _stream()),
         "attn_decode_units")
     global LAUNCHES, BY_LENGTH_CALLS
     BY_LENGTH_CALLS += 1
@@ -720,13 +746,13 @@ def attn_decode_units(q, q_stride, pages, table, cu_q, ctx_lens, n_seqs, out, pa
 
 def paged_attention(q: torch.Tensor, q_stride: int, pages: torch.Tensor, table: torch.Tensor, ctx,
                     out: torch.Tensor, nq: int, nkv: int, d: int, scale: float, window: int,
-                    dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0, sink: bool = False) -> None:
+                    dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0, sink: Sink = None) -> None:
     """Attention of a step's tokens over the paged cache; picks the kernel: the
     tensor-core kernels for bfloat16 and head sizes in steps of 16, the plain
     kernel for 32-bit and every other head size up to 256.  ``dist_bias`` float32 [nq, L >= window]: entry
     (h, i - j) is taken off the score of query position i and key position j.  ``softcap`` c > 0: the scaled score s
-    becomes c tanh(s / c), before the bias.  ``sink``: one more entry in the softmax's denominator, of score 0 and without a
-    value."""
+    becomes c tanh(s / c), before the bias.  ``sink`` float32 [nq] (or True: zeros): one more entry in every softmax's
+    denominator, of the head's score and without a value."""
     if _ATTN_FORCE_SIMT or not mma_attention_supported(q.dtype, d):
         paged_attention_simt(q, q_stride, pages, table, ctx.token_seq, ctx.positions, out, nq, nkv, d,
                              scale, window, ctx.status, dist_bias, softcap, sink)
@@ -736,7 +762,8 @@ def paged_attention(q: torch.Tensor, q_stride: int, pages: torch.Tensor, table: 
     n_dec = ctx.num_decode_seqs if G <= 16 else 0      # these come first in the step's arrays
     if n_dec:
         # one-token sequences: split-KV kernel
-        splits = decode_splits(n_dec, nkv, ctx.max_kv_len)
+        # a window or a chunk bounds the keys a query walks, however long its sequence is
+        splits = decode_splits(n_dec, nkv, min(ctx.max_kv_len, abs(window)) if window else ctx.max_kv_len)
         units = decode_units(n_dec, nkv, d, ctx.ranges_by_length)
         part_o, part_ml, seq_ranges = _decode_scratch(ctx.workspace, n_dec, nq, nkv, d, splits)
         if units:
@@ -757,16 +784,18 @@ def paged_attention(q: torch.Tensor, q_stride: int, pages: torch.Tensor, table: 
                 memo[("attn_tail", id(table), n_dec)] = tail
         table_t, cu_q_t, ctx_lens_t = tail
         if USE_TC_ATTENTION and tc_attention_supported(q.dtype, d, pages.shape[3], ctx.max_kv_len):
-            plan = memo.get(("attn_tc_plan", G, nkv, n_dec, ctx.captured)) if memo is not None else None
+            plan = memo.get(("attn_tc_plan", G, nkv, n_dec, ctx.captured, window)) if memo is not None else None
             if plan is None:
                 tiles = sum(-(-(ql * G) // 128) for ql in ctx.q_lens[n_dec:])
                 # a captured step does not know its requests' lengths: the level it was captured for stands in
                 key_tiles = 4 * getattr(ctx, "key_share_level", 0) if ctx.captured else \
                     max(-(-(c + ql) // 64) for c, ql in zip(ctx.ctx_lens_host[n_dec:], ctx.q_lens[n_dec:]))
+                if window:                       # a row tile's tokens and the keys in front of the first of them
+                    key_tiles = min(key_tiles, (abs(window) + 128 // G) // 64 + 2)
                 count = attn_tc_shares(tiles, nkv, key_tiles)
                 plan = (tiles, count, sum(ctx.q_lens[:n_dec]), sum(ctx.q_lens[n_dec:]))
                 if memo is not None:
-                    memo[("attn_tc_plan", G, nkv, n_dec, ctx.captured)] = plan
+                    memo[("attn_tc_plan", G, nkv, n_dec, ctx.captured, window)] = plan
             tiles, count, row0, rows = plan
             shares = None
             if count > 1:
@@ -965,24 +994,27 @@ def moe_row_tile(tensor_cores: bool) -> int:
     return int(_lib("moe").ff_moe_row_tile(c_int(1 if tensor_cores else 0)))
 
 
-ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1            # how router logits become scores
+ROUTE_SOFTMAX, ROUTE_SIGMOID, ROUTE_CHOSEN_SOFTMAX = 0, 1, 2   # how router logits become scores (and weights)
 GROUP_BY_BEST, GROUP_BY_TWO_BEST = 0, 1        # a group's score: its largest choice score, or the sum of its two largest
 GLU_CLAMPED_SWISH, GLU_SILU = 0, 1             # an expert's activation (gated experts)
 MOE_DOWN, MOE_GATE_UP, MOE_UP = 0, 1, 2        # the grouped products: second one, first one of gated / ungated experts
 
 
 def moe_route(z, ids, wts, groups: int, keep: int, *, score: int = ROUTE_SOFTMAX, correction=None,
-              group_score: int = GROUP_BY_BEST, renormalize: bool = True) -> None:
+              group_score: int = GROUP_BY_BEST, renormalize: bool = True, bias=None) -> None:
     """Choice of experts per token from router logits z float32 [T,E] (rows may be the head of wider ones): ids int32 [T,top], wts float32 [T,top].
+    ``bias`` float32 [E] is added to the logits.  ROUTE_CHOSEN_SOFTMAX: chosen by the logits, the weights are the softmax over
+    the chosen ones alone.
     ``correction`` float32 [E]: added to the scores for the choice only (the weights are the plain scores)."""
-    _need_cuda(ids, wts, correction)
+    _need_cuda(ids, wts, correction, bias)
     if not z.is_cuda or z.stride(1) != 1:
         raise KernelError("moe_route: the logits must be a CUDA matrix with contiguous rows")
     T, E = z.shape
     top = ids.shape[1]
     assert z.dtype == torch.float32 and ids.dtype == torch.int32 and wts.dtype == torch.float32 and wts.shape == ids.shape
-    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
-    _check(_lib("moe").ff_moe_route(_p(z), c_int(z.stride(0)), _p(correction), c_int(T), c_int(E), c_int(top), c_int(groups), c_int(keep),
+    for extra in (correction, bias):
+        assert extra is None or (extra.dtype == torch.float32 and extra.numel() == E)
+    _check(_lib("moe").ff_moe_route(_p(z), c_int(z.stride(0)), _p(bias), _p(correction), c_int(T), c_int(E), c_int(top), c_int(groups), c_int(keep),
                                    c_int(score), c_int(group_score), c_int(1 if renormalize else 0), _p(ids), _p(wts),
                                    _stream()), "moe_route")
 
@@ -1108,15 +1140,61 @@ def scale_(x: torch.Tensor, a: float) -> None:
     _check(_lib("elementwise").ff_scale(_p(x), c_float(a), c_size_t(x.numel()), _stream()), "scale")
 
 
+def softcap_(x: torch.Tensor, cap: float) -> None:
+    """x <- cap * tanh(x / cap) for a contiguous float32 tensor."""
+    _need_cuda(x)
+    assert x.dtype == torch.float32 and x.is_contiguous() and cap > 0
+    _check(_lib("elementwise").ff_softcap(_p(x), c_float(cap), c_size_t(x.numel()), _stream()), "softcap")
+
+
+def stream_seam(src: torch.Tensor, out: torch.Tensor, *, streams: int, y: Optional[torch.Tensor] = None, routed=None, mix=None,
+                out_w=None, in_w=None, dst: Optional[torch.Tensor] = None, w=None, b=None, eps: float = 0.0, center: bool = True,
+                row_idx: Optional[torch.Tensor] = None) -> None:
+    """The seam between two parts of a model with ``streams`` = S residual streams.  ``src`` float32 [T, S, W], or [T, W]
+    when all streams are equal.  With ``y`` [T, W] (float32 or bfloat16), or ``routed`` = (rows float32, row_of int32 [T top],
+    wts float32 [T, top], shared float32 [T, W] or None), which stands for y[t] = sum_k wts[t, k] rows[row_of[t, k]] +
+    shared[t], the streams first become x_t <- sum_s mix[s, t] x_s + out_w[t] y (kept in ``dst``, which may be ``src``, unless
+    it is None).  Then u = sum_s in_w[s] x_s (``in_w`` None: the plain sum) and out = norm(u) * w + b with ``center`` a layer
+    norm, else an RMS norm; ``w`` None: out = u.  ``row_idx`` int32: only these tokens' rows, into out's rows."""
+    rows = row_of = wts = shared = None
+    if routed is not None:
+        rows, row_of, wts, shared = routed
+    _need_cuda(src, out, y, rows, row_of, wts, shared, mix, out_w, in_w, dst, w, b, row_idx)
+    S, same = int(streams), src.dim() == 2
+    T, W = src.shape[0], src.shape[-1]
+    assert src.dtype == torch.float32 and (same or src.shape[1] == S) and out.dim() == 2 and out.shape[1] == W
+    kind = 0
+    if routed is not None:
+        assert y is None and rows.dtype == wts.dtype == torch.float32 and rows.shape[1] == W and wts.shape[0] == T
+        assert row_of.dtype == torch.int32 and row_of.numel() >= wts.numel()
+        assert shared is None or (shared.dtype == torch.float32 and shared.shape == (T, W))
+        kind = 3
+    elif y is not None:
+        assert y.shape == (T, W)
+        kind = 1 + _dt(y)
+    for t, n in ((mix, S * S), (out_w, S), (in_w, S), (w, W), (b, W)):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == n)
+    assert kind == 0 or (mix is not None and out_w is not None)
+    assert dst is None or (dst.dtype == torch.float32 and dst.shape == (T, S, W) and kind != 0 and row_idx is None)
+    assert row_idx is None or row_idx.dtype == torch.int32
+    n = T if row_idx is None else row_idx.numel()
+    assert out.shape[0] == n
+    _check(_lib("stream_seam").ff_stream_seam(
+        _p(src), _p(dst), _p(y), c_int(kind), _p(rows), _p(row_of), _p(wts), c_int(wts.shape[1] if wts is not None else 0),
+        _p(shared), _p(mix), _p(out_w), _p(in_w), _p(w), _p(b), c_float(eps), c_int(1 if center else 0), _p(out),
+        c_int(_dt(out)), _p(row_idx), c_int(n), c_int(S), c_int(W), c_int(1 if same else 0), _stream()), "stream_seam")
+
+
 def head_finish(qkv: torch.Tensor, nq: int, nkv: int, d: int, norm_dim: int, eps: float, freq: Optional[torch.Tensor],
                 mag: float, ctx, block_table: Optional[torch.Tensor], cache: Optional[torch.Tensor], *,
                 interleaved: bool = False, normalize: bool = False, bias: Optional[torch.Tensor] = None,
                 q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None, q_temp=None,
-                value_is_key: bool = False) -> None:
+                value_is_key: bool = False, norm_all: bool = False) -> None:
     """Finish the heads of the projection's rows ``qkv`` [T, >= (nq + 2 nkv) d]: q goes back in place, k and v into the paged
     cache [blocks, 2, nkv, block, d] (``nkv == 0``: q only).  In this order, each optional: ``bias`` float32 in the row's
-    layout; an RMS norm of each q / k head over ``norm_dim`` elements with weights ``q_norm_w`` / ``k_norm_w`` float32 [d];
-    the rotation of the first 2 * len(freq) elements (angle = position * freq, formed in 64-bit; cos and sin times ``mag``;
+    layout; an RMS norm of each q / k head over ``norm_dim`` elements with weights ``q_norm_w`` / ``k_norm_w`` float32 [d]
+    (``norm_all``: one norm over all q heads together and one over all k heads, weights [nq d] / [nkv d], a head counting
+    ``norm_dim`` elements); the rotation of the first 2 * len(freq) elements (angle = position * freq, formed in 64-bit; cos and sin times ``mag``;
     ``interleaved``: element 2i turns with element 2i + 1, else i with i + len(freq)); ``normalize``: q and k divided by
     their root mean square over ``norm_dim`` elements; ``q_temp`` = (coef, every): q times
     1 + coef ln(floor((position + 1) / every) + 1).  ``value_is_key``: a row is q | k, and the value is k as projected."""
@@ -1126,8 +1204,8 @@ def head_finish(qkv: torch.Tensor, nq: int, nkv: int, d: int, norm_dim: int, eps
     assert width >= need and (freq is None or freq.dtype == torch.float64)
     if bias is not None:
         assert bias.dtype == torch.float32 and bias.numel() == need and bias.is_contiguous()
-    for w in (q_norm_w, k_norm_w):
-        assert w is None or (w.dtype == torch.float32 and w.numel() == d)
+    for w, n in ((q_norm_w, nq), (k_norm_w, nkv)):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == (n * d if norm_all else d) and w.is_contiguous())
     if nkv:
         num_blocks, two, ckv, block_size, cd = cache.shape
         assert two == 2 and ckv == nkv and cd == d and cache.dtype == qkv.dtype
@@ -1139,7 +1217,7 @@ def head_finish(qkv: torch.Tensor, nq: int, nkv: int, d: int, norm_dim: int, eps
         _p(freq), c_int(2 * freq.numel() if freq is not None else 0), c_float(mag), _p(ctx.positions), _p(ctx.token_seq),
         _p(block_table), c_int(max_blocks), c_int(block_size), c_int(num_blocks), _p(cache), _p(ctx.status),
         c_int(1 if interleaved else 0), c_int(1 if normalize else 0), _p(bias), _p(q_norm_w), _p(k_norm_w),
-        *_temp_args(q_temp), c_int(1 if value_is_key else 0), _stream()), "head_finish")
+        *_temp_args(q_temp), c_int(1 if value_is_key else 0), c_int(1 if norm_all else 0), _stream()), "head_finish")
 
 
 def rope_unit_norm_store(qkv, nq: int, nkv: int, d: int, norm_dim: int, eps: float, freq: torch.Tensor, mag: float, ctx,

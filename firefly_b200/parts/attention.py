@@ -33,6 +33,9 @@ Further parameters, for designs that differ from the above (defaults: as above):
                     finishes the heads
     softcap         c > 0: the scaled score s becomes c tanh(s / c)
     sink            True: one more entry in every softmax's denominator, of score 0 and without a value
+    sink_leaf       the tensor [num_heads] of such an entry's score, a number a head (not scaled)
+    qk_norm_over    "head" (default) or "all": with ``qk_norm`` one norm over all query heads together and one over all key
+                    heads, weights [num_heads * head_dim] and [num_kv_heads * head_dim]
     value_is_key    True: there is no W_v; the values are the keys as projected (before norm and rotation)
     q_temp          (coef, every): q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)
     gate_leaf       the tensor [num_heads, hidden] of one output gate a head: head h's output is multiplied by
@@ -87,6 +90,12 @@ class GQAttention(Part):
         if self.softcap < 0:
             raise ValueError("softcap must be positive (or absent)")
         self.sink = bool(self.p("sink", False))
+        self.sink_leaf = self.p("sink_leaf", None)
+        self.sinks = None                                 # float32 [num_heads] once bound
+        over = str(self.p("qk_norm_over", "head"))
+        if over not in ("head", "all") or (over == "all" and not self.qk_norm):
+            raise ValueError("qk_norm_over is 'head' or, with qk_norm, 'all'")
+        self.norm_all = over == "all"
         self.value_is_key = bool(self.p("value_is_key", False))
         q_temp = self.p("q_temp", None)
         self.q_temp = None if q_temp is None else (float(q_temp[0]), int(q_temp[1]))
@@ -102,7 +111,7 @@ class GQAttention(Part):
         no_table = position is not None and hasattr(position, "frequencies") and getattr(position, "max_positions", 1) == 0
         # the kernel that forms the angles from the frequencies also adds biases, takes either pairing, a temperature, ...
         self.by_frequencies = self.unit_norm or interleaved or self.bias_suffix is not None or no_table \
-            or self.q_temp is not None or self.value_is_key or (self.qk_norm and self.dk != self.d)
+            or self.q_temp is not None or self.value_is_key or (self.qk_norm and self.dk != self.d) or self.norm_all
         if self.by_frequencies and position is not None and not hasattr(position, "frequencies"):
             raise ValueError("this attention needs a position encoding that gives its frequencies")
         self.interleaved = interleaved
@@ -145,7 +154,10 @@ class GQAttention(Part):
                           [WeightSpec(self.name(L["v"]) + sfx, (self.nkv * self.dv,), init="zeros", as_float32=True)])]
         if self.qk_norm:
             for kind in ("q", "k") if self.has_kv else ("q",):
-                out.append(WeightSpec(self.name(self.norm_leaf[kind]), (self.dk,), init="norm", as_float32=True))
+                heads = (self.nq if kind == "q" else self.nkv) if self.norm_all else 1
+                out.append(WeightSpec(self.name(self.norm_leaf[kind]), (heads * self.dk,), init="norm", as_float32=True))
+        if self.sink_leaf is not None:
+            out.append(WeightSpec(self.name(self.sink_leaf), (self.nq,), init="zeros", as_float32=True))
         return out
 
     def fused_layout(self, dtype_of) -> List[FusedSpec]:
@@ -207,6 +219,10 @@ class GQAttention(Part):
                 full[:, :size] = b
                 rows.append(full.view(-1))
             self.bias = torch.cat(rows).contiguous()
+        if self.sink_leaf is not None:
+            self.sinks = self._vector32(tensors[self.name(self.sink_leaf)])
+        elif self.sink:
+            self.sinks = torch.zeros((self.nq,), dtype=torch.float32, device=self.w_o.device)
         if self.qk_norm:
             self.q_norm_w = self._norm_row(tensors, "q")
             if self.has_kv:
@@ -216,9 +232,10 @@ class GQAttention(Part):
         w = self._vector32(tensors[self.name(self.norm_leaf[kind])])
         if self.dk == self.d:
             return w
-        full = torch.zeros((self.d,), dtype=torch.float32, device=w.device)       # a head that is filled up with zeros
-        full[: self.dk] = w
-        return full
+        w = w.view(-1, self.dk)                                                   # one head's weights, or every head's
+        full = torch.zeros((w.shape[0], self.d), dtype=torch.float32, device=w.device)      # heads filled up with zeros
+        full[:, : self.dk] = w
+        return full.view(-1)
 
     # -- run ------------------------------------------------------------------
     def _mask(self) -> int:
@@ -255,12 +272,12 @@ class GQAttention(Part):
         att = ws.get("attn.out", (T, self.nq * self.d), ctx.dtype)
         turns = self.position is not None and hasattr(self.position, "frequencies")
         if write_cache and self.chunk is None and not self.softcap and self.dk == self.d and not self.unit_norm \
-                and self.bias is None and not (self.by_frequencies and turns) and (self.qk_norm or self.q_temp is None) \
+                and self.bias is None and not self.norm_all and not (self.by_frequencies and turns) and (self.qk_norm or self.q_temp is None) \
                 and K.decode_finishes_heads(ctx, ctx.dtype, self.nq, self.nkv, self.d, rotary_dim):
             # a step of single tokens: the attention kernel finishes the heads itself
             K.attn_decode_heads(qkv, pages, table, ctx, att, self.nq, self.nkv, self.d, self.scale,
                                 0 if self.window is None else int(self.window), self.q_norm_w,
-                                self.k_norm_w, self.eps, cos_sin, sink=self.sink, q_temp=self.q_temp,
+                                self.k_norm_w, self.eps, cos_sin, sink=self.sinks, q_temp=self.q_temp,
                                 value_is_key=self.value_is_key)
         elif self.by_frequencies:
             freq, mag = (self.position.frequencies(), self.position.magnitude) if turns else (None, 1.0)
@@ -269,7 +286,7 @@ class GQAttention(Part):
                           table if write_cache else None, pages if write_cache else None,
                           interleaved=self.interleaved, normalize=self.unit_norm, bias=bias, q_norm_w=self.q_norm_w,
                           k_norm_w=self.k_norm_w if write_cache else None, q_temp=self.q_temp,
-                          value_is_key=self.value_is_key)
+                          value_is_key=self.value_is_key, norm_all=self.norm_all)
             self._attend(qkv, width, pages, table, ctx, att)
         else:
             K.qk_norm_rope_store(qkv, self.nq, nkv_w, self.d, self.q_norm_w,
@@ -287,7 +304,7 @@ class GQAttention(Part):
 
     def _attend(self, qkv, width, pages, table, ctx, att) -> None:
         K.paged_attention(qkv, width, pages, table, ctx, att, self.nq, self.nkv, self.d, self.scale,
-                          self._mask(), softcap=self.softcap, sink=self.sink)
+                          self._mask(), softcap=self.softcap, sink=self.sinks)
 
 
 register_part("mixer", "gqa_attention", GQAttention)

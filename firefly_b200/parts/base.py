@@ -47,6 +47,9 @@ folds_next_norm         forward(then_norm=)         ... and, told which norm fol
 scales_residual         forward(residual_scale=)    ... and adds it times a constant (a block whose parts'
                                                     outputs enter the stream times a multiplier)
 accepts_folded_norm     (none)                      its first operation can finish a ``FoldedNorm``
+hands_on_rows           forward(as_rows=)           feed_forward: may return its routed experts' rows with their
+                                                    weights (``RoutedRows``), whose sum the block forms on its way
+                                                    into the stream
 hands_on_normed_sum     forward(as_sum=)            mixer: may return its result as a ``NormedSum`` that the
                                                     block's norm forms on its way into the stream
 takes_next_norm         forward(next_norm=)         arrangement: hands the next block's first norm
@@ -94,7 +97,7 @@ def part_class(category: str, kind: str) -> type:
 
 _FLAG_KEYWORD = {"adds_into_residual": "accumulate_into", "folds_next_norm": "then_norm",
                  "takes_next_norm": "next_norm", "scales_residual": "residual_scale",
-                 "hands_on_normed_sum": "as_sum"}
+                 "hands_on_normed_sum": "as_sum", "hands_on_rows": "as_rows"}
 _FLAG_MEMBERS = {"foldable": ("fold_buffers", "size", "eps")}
 
 
@@ -149,6 +152,7 @@ class Part:
     accepts_folded_norm = False
     foldable = False
     hands_on_normed_sum = False
+    hands_on_rows = False
 
     def __init__(self, spec: PartSpec, rt: Runtime):
         self.spec = spec

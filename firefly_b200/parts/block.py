@@ -86,9 +86,11 @@ class Block:
         return self.input_filter.forward(x, ctx, ctx.memo["filter_slot"])
 
     def weight_specs(self) -> List[WeightSpec]:
-        # ``params["unused_vectors"]``: (name, size) of vectors that a checkpoint may hold for a half the block does not have
+        # ``params["unused_vectors"]``: (name, size or shape) of tensors that a checkpoint may hold for a half the block does
+        # not have
         return [w for p in self.parts() for w in p.weight_specs()] + \
-            [WeightSpec(name, (int(size),), as_float32=True, optional=True) for name, size in self.params.get("unused_vectors", ())]
+            [WeightSpec(name, tuple(size) if isinstance(size, (tuple, list)) else (int(size),), as_float32=True, optional=True)
+             for name, size in self.params.get("unused_vectors", ())]
 
     takes_next_norm = False      # an arrangement whose forward takes ``next_norm`` sets this
 

@@ -51,6 +51,9 @@ class LMHead(Part):
         self.tied_to = self.p("tied_to", None)
         self.tensor = self.p("tensor", None) or self.name("weight")   # full tensor name, if it is not <prefix>.weight
         self.scale = float(self.p("scale", 1.0))                      # the logits times this, in 32-bit
+        self.softcap = float(self.p("softcap", 0.0) or 0.0)           # c > 0: then c tanh(logit / c), in 32-bit
+        if self.softcap < 0:
+            raise ValueError("softcap must be positive (or absent)")
         self.weight = None
 
     def weight_specs(self) -> List[WeightSpec]:
@@ -68,6 +71,8 @@ class LMHead(Part):
             apply_linear(x_rows, self.weight, out, ctx, "logits")
             if self.scale != 1.0:
                 K.scale_(out, self.scale)
+            if self.softcap:
+                K.softcap_(out, self.softcap)
         return out
 
 

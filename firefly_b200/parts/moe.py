@@ -19,6 +19,8 @@ shared.gate, shared.up [shared_ff, W]; shared.down [W, shared_ff].
 
 What the lines above fix can be chosen by further parameters (the defaults are the above):
     score          "softmax" | "sigmoid": s = sigmoid(z), each expert by itself
+                   | "chosen_softmax": the choice is by z itself and the weights are the softmax over the chosen z alone
+    router_bias    the leaf of a tensor [experts] added to z (None: none)
     correction     True: a tensor ``correction`` [experts] is added to s for the choice (of groups and of experts);
                    the weights stay the plain s
     group_score    "best" | "two_best": a group's score is the sum of its two largest choice scores
@@ -44,8 +46,16 @@ from .base import Part, register_part
 from .linear import apply_linear, linear_relu2
 
 
+class RoutedRows:
+    """A step's routed output that has not been summed: token t's is sum_k wts[t, k] rows[row_of[t, k]] + shared[t]."""
+
+    def __init__(self, rows: torch.Tensor, row_of: torch.Tensor, wts: torch.Tensor, shared):
+        self.rows, self.row_of, self.wts, self.shared = rows, row_of, wts, shared
+
+
 class GroupedExperts(Part):
     adds_into_residual = True        # forward(accumulate_into=...)
+    hands_on_rows = True             # forward(as_rows=...)
     scales_residual = True           # forward(residual_scale=...)
 
     def __init__(self, spec, rt):
@@ -62,11 +72,13 @@ class GroupedExperts(Part):
         self.limit = float(self.p("limit", 0.0 if act != "clamped_swish" else ...))
         self.weight_on_input = bool(self.p("weight_on_input", False))
         self.shared_gate = bool(self.p("shared_gate", False))
-        self.score = {"softmax": K.ROUTE_SOFTMAX, "sigmoid": K.ROUTE_SIGMOID}[str(self.p("score", "softmax"))]
+        self.score = {"softmax": K.ROUTE_SOFTMAX, "sigmoid": K.ROUTE_SIGMOID, "chosen_softmax": K.ROUTE_CHOSEN_SOFTMAX}[str(self.p("score", "softmax"))]
         self.group_score = {"best": K.GROUP_BY_BEST, "two_best": K.GROUP_BY_TWO_BEST}[str(self.p("group_score", "best"))]
         self.renormalize = bool(self.p("renormalize", True))
         self.has_correction = bool(self.p("correction", False))
         self.correction = None
+        self.router_bias_leaf = self.p("router_bias", None)
+        self.router_bias = None
         self.shared_ff = int(self.p("shared_ff", 0))
         self.shared_limit = float(self.p("shared_limit", self.limit))
         if self.E % self.groups or not (0 < self.keep <= self.groups) or not (0 < self.top <= self.keep * (self.E // self.groups)):
@@ -80,6 +92,8 @@ class GroupedExperts(Part):
     def weight_specs(self) -> List[WeightSpec]:
         n, W = self.name, self.hidden
         out = [WeightSpec(n("router"), (self.E, W))]
+        if self.router_bias_leaf is not None:
+            out.append(WeightSpec(n(self.router_bias_leaf), (self.E,), init="zeros", as_float32=True))
         if self.has_correction:
             out.append(WeightSpec(n("correction"), (self.E,), init="zeros", as_float32=True))
         for e in range(self.E):
@@ -122,6 +136,8 @@ class GroupedExperts(Part):
         E, W = self.E, self.hidden
         self.router = self._stacked(tensors, "router_sg", ["router", "shared.sg"]) if self.shared_gate \
             else self._matrix(tensors[self.name("router")])
+        if self.router_bias_leaf is not None:
+            self.router_bias = self._vector32(tensors[self.name(self.router_bias_leaf)])
         if self.has_correction:
             self.correction = self._vector32(tensors[self.name("correction")])
         if self.gated:
@@ -136,7 +152,7 @@ class GroupedExperts(Part):
                 else self._matrix(tensors[self.name("shared.up")])
             self.w_sh_down = self._matrix(tensors[self.name("shared.down")])
 
-    def forward(self, x, ctx, accumulate_into=None, residual_scale: float = 1.0):
+    def forward(self, x, ctx, accumulate_into=None, residual_scale: float = 1.0, as_rows: bool = False):
         T, ws, W, top = x.shape[0], ctx.workspace, self.hidden, self.top
         dt = self.w_up.dtype
         if x.dtype != dt:
@@ -147,7 +163,7 @@ class GroupedExperts(Part):
         ids = ws.get("moe.ids", (T, top), torch.int32)
         wts = ws.get("moe.wts", (T, top), torch.float32)
         K.moe_route(z[:, : self.E], ids, wts, self.groups, self.keep, score=self.score, correction=self.correction,
-                    group_score=self.group_score, renormalize=self.renormalize)
+                    group_score=self.group_score, renormalize=self.renormalize, bias=self.router_bias)
         rows = T * top
         tc = K.moe_on_tensor_cores(dt, (W, self.ff))       # which grouped kernel runs: the plan's row tile is its
         max_tiles = K.moe_max_tiles(rows, self.E, tc)
@@ -178,6 +194,8 @@ class GroupedExperts(Part):
                 linear_relu2(x, self.w_sh_gu, sact, ctx, "moe.sh_up")
             shared = ws.get("moe.sh_out", (T, W), torch.float32)
             apply_linear(sact, self.w_sh_down, shared, ctx, "moe.sh_out")
+        if as_rows and accumulate_into is None and not self.weight_on_input and not self.shared_gate:
+            return RoutedRows(outs, row_of, wts, shared)
         into = accumulate_into if accumulate_into is not None else ws.get("moe.delta", (T, W), torch.float32)
         K.moe_combine(into, outs, row_of, None if self.weight_on_input else wts, shared, residual_scale if accumulate_into is not None else 1.0,
                       top=top, shared_z=z[:, self.E] if self.shared_gate else None, overwrite=accumulate_into is None)
