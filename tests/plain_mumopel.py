@@ -181,9 +181,9 @@ def random_weights(cfg: Mapping, seed: int) -> Dict[str, torch.Tensor]:
         H, G, d, dv = (int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
         for q in (1, 2) if ml is not None else (1,):
             w[f"{p}.norm{q}"], w[f"{p}.norm{q}.b"] = rnd(W, std=0.2, mean=1.0), rnd(W, std=0.1)
-            w[f"{p}.hc{q}.in"], w[f"{p}.hc{q}.out"] = rnd(S, std=0.5, mean=1.0 / S), rnd(S, std=0.5, mean=0.7)
+            w[f"{p}.hc{q}.in"], w[f"{p}.hc{q}.out"] = rnd(S, std=0.3 / S, mean=1.0 / S), rnd(S, std=0.25, mean=0.5)
             # not symmetric, every stream fed by every other, and a size that neither dies nor grows over the layers
-            w[f"{p}.hc{q}.mix"] = (0.75 * torch.eye(S, dtype=torch.float64) + rnd(S, S, std=0.3 / math.sqrt(S))).to(torch.bfloat16).double()
+            w[f"{p}.hc{q}.mix"] = (0.8 * torch.eye(S, dtype=torch.float64) + rnd(S, S, std=0.1, mean=0.2 / S)).to(torch.bfloat16).double()
         a = p + ".mix"
         w[a + ".q"], w[a + ".k"], w[a + ".v"], w[a + ".o"] = lin(H * d, W), lin(G * d, W), lin(G * dv, W), lin(W, H * dv)
         w[a + ".q.norm"], w[a + ".k.norm"] = rnd(H * d, std=0.3, mean=1.0), rnd(G * d, std=0.3, mean=1.0)
@@ -195,7 +195,7 @@ def random_weights(cfg: Mapping, seed: int) -> Dict[str, torch.Tensor]:
             [(f"{f}.e{e}", int(ml["expert"]["ff"])) for e in range(int(ml["router"]["experts"]))] + \
             ([(f + ".shared", int(ml["shared"]["ff"]))] if ml.get("shared") else [])
         for n, F in names:
-            w[n + ".gate"], w[n + ".up"], w[n + ".down"] = lin(F, W, 1.5), lin(F, W, 1.5), lin(W, F)
+            w[n + ".gate"], w[n + ".up"], w[n + ".down"] = lin(F, W, 1.2), lin(F, W, 1.2), lin(W, F, 0.7)
         if ml["kind"] == "moe":
             E = int(ml["router"]["experts"])
             w[f + ".router"], w[f + ".router.b"] = lin(E, W), rnd(E, std=0.7)
