@@ -1,7 +1,7 @@
 """Throughput of a design beside the closest existing model at equal size: Kolorax beside Qwen3 dense, Pepolorn
-beside Kolorax, Kefisun beside Qwen3 dense, Papusun beside Kefisun, Gatutar beside Pepolorn.
+beside Kolorax, Kefisun beside Qwen3 dense, Papusun beside Kefisun, Gatutar beside Pepolorn, Mumopel beside Qwen3 dense.
 
-``python bench.py --design kolorax`` (or ``pepolorn``, ``kefisun``, ``papusun``, ``gatutar``) calls `main` here; the default workload of bench.py is untouched.
+``python bench.py --design kolorax`` (or ``pepolorn``, ``kefisun``, ``papusun``, ``gatutar``, ``mumopel``) calls `main` here; the default workload of bench.py is untouched.
 For each size, both models are built with seeded random weights at layer sizes that resemble a real
 model's (same width, same number of layers, the dense feed-forward as wide as the experts a token
 uses plus the shared one) and run through the engine's own loop (`Engine`: scheduler, captured decode
@@ -296,6 +296,8 @@ def main(args, peaks: dict) -> int:
         return papusun_main(args, peaks)
     if args.design == "gatutar":
         return gatutar_main(args, peaks)
+    if args.design == "mumopel":
+        return mumopel_main(args, peaks)
     out = {"design": "Kolorax", "beside": "Qwen3 dense at equal width, layers and feed-forward width per token",
            "dtype": args.dtype, "batch": args.batch, "prompt_len": args.prompt_len, "new_tokens": args.steps,
            "data": "synthetic token ids, seeded random weights", "peaks": peaks.get("source"), "sizes": {}}
@@ -881,6 +883,139 @@ def gatutar_main(args, peaks: dict) -> int:
         beside = run_engine(pepolorn_config(**shape), args.dtype, args.batch, args.prompt_len, args.steps)
         out["sizes"][name] = {"shape": shape, "gatutar": ours, "pepolorn": beside,
                               "kernels": gatutar_kernel_table(size["width"], size["ff"], args.batch, args.prompt_len, peaks)}
+        print(json.dumps({"partial": name, **out["sizes"][name]}), flush=True)
+    print(json.dumps(out))
+    return 0
+
+
+# --------------------------------------------------------------------------- #
+# Mumopel beside Qwen3 dense
+MUMOPEL_STREAMS, MUMOPEL_CHUNK = 4, 8192
+
+
+def mumopel_config(width: int, layers: int, ff: int, shared_ff: int) -> dict:
+    """Every layer attention in long chunks (heads of 128, four query heads a kv head, half of a head rotated, a sink a
+    head) over four streams; the first feed-forward dense, the others four of sixteen experts and a shared one."""
+    heads = width // 128
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": MUMOPEL_CHUNK},
+           "rot": {"base": 10000.0, "dims": 64}}
+    moe = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": ff, "limit": 7.0}, "shared": {"ff": shared_ff, "limit": 7.0}}
+    return {"architecture": "Mumopel", "vocab": VOCAB, "width": width, "streams": MUMOPEL_STREAMS, "logit_softcap": 30.0, "norm": {"eps": 1e-6},
+            "layers": [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": TOP * ff + shared_ff} if i == 0 else moe}
+                       for i in range(layers)]}
+
+
+def mumopel_kernel_table(width: int, ff: int, batch: int, prompt: int, peaks: dict) -> list:
+    """The kernels that Mumopel added or changed, alone against their floors, each beside the like kernel (or the same
+    kernel without the new option) of the models that were there."""
+    from .ops import kernels as K
+    dev = torch.device("cuda:0")
+    bf = torch.bfloat16
+    flush = torch.empty(192 << 20, dtype=torch.uint8, device=dev)
+    hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    rows = []
+
+    def add(name, us, bytes_=0, flops=0, like=None):
+        floor = max(bytes_ / hbm, flops / tflops) * 1e6
+        rows.append({"kernel": name, "us": round(us, 1), "floor_us": round(floor, 2), "of_floor": round(floor / us, 3) if us else None,
+                     "bound": "memory" if bytes_ / hbm >= flops / tflops else "tensor", "like": like})
+    H, d, block, S = width // 128, 128, 16, MUMOPEL_STREAMS
+    G = max(1, H // 4)
+    for label, n_seqs, q, ctx_len in (("prefill", batch, prompt, 0), ("decode", batch * 8, 1, prompt)):
+        T = n_seqs * q
+        per = -(-(q + ctx_len) // block)
+        ctx = SimpleNamespace(cu_q=torch.arange(0, T + 1, q, dtype=torch.int32, device=dev), num_seqs=n_seqs,
+                              token_seq=torch.arange(T, dtype=torch.int32, device=dev) // q,
+                              positions=(torch.arange(T, dtype=torch.int32, device=dev) % q) + ctx_len,
+                              status=torch.zeros(1, dtype=torch.int32, device=dev), workspace=_Scratch(dev))
+        ctx_lens = torch.full((n_seqs,), ctx_len, dtype=torch.int32, device=dev)
+        table = (torch.arange(n_seqs * per, dtype=torch.int32, device=dev) + 1).view(n_seqs, per).contiguous()
+        pages = (torch.randn(n_seqs * per + 1, 2, G, block, d, device=dev) * 0.5).to(bf)
+        # -- heads finished: one norm over all heads, a norm a head, rotation only
+        C = (H + 2 * G) * d
+        qkv = (torch.randn(T, C, device=dev) * 0.5).to(bf)
+        freq = torch.pow(torch.tensor(10000.0, dtype=torch.float64), -torch.arange(32, dtype=torch.float64) / 32).to(dev)
+        qw, kw = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+        us = _time(lambda: K.head_finish(qkv, H, G, d, d, 1e-6, freq, 1.0, ctx, table, pages, interleaved=True, q_norm_w=qw, k_norm_w=kw,
+                                         norm_all=True), flush=flush)
+        add(f"head finish: one norm over all heads, rotation {label} ({T} rows)", us, T * C * 2 * 2, like="head finish: a norm a head, rotation")
+        us = _time(lambda: K.head_finish(qkv, H, G, d, d, 1e-6, freq, 1.0, ctx, table, pages, interleaved=True, q_norm_w=qw[:d], k_norm_w=kw[:d]),
+                   flush=flush)
+        add(f"head finish: a norm a head, rotation {label} ({T} rows)", us, T * C * 2 * 2)
+        # -- attention with a sink a head in chunks, and plain
+        att = torch.empty(T, H * d, dtype=bf, device=dev)
+        sinks = torch.zeros(H, device=dev)
+        if q > 1:
+            flops = 4 * n_seqs * (q * (q + 1) // 2) * H * d
+            tiles = n_seqs * -(-(q * (H // G)) // 128)
+            for name, sink, mask in (("attention tcgen05, sinks, chunks", sinks, -MUMOPEL_CHUNK), ("attention tcgen05", None, 0)):
+                us = _time(lambda: K.attn_tc(qkv, C, pages, table, ctx.cu_q, ctx_lens, n_seqs, tiles, att, H, G, d, d ** -0.5, mask,
+                                             ctx.status, sink=sink), flush=flush)
+                add(f"{name} {label}", us, T * (2 * H + 2 * G) * d * 2, flops, like="attention tcgen05" if mask else None)
+            small = 256                                                          # chunks that bind: what is outside is not walked
+            us = _time(lambda: K.attn_tc(qkv, C, pages, table, ctx.cu_q, ctx_lens, n_seqs, tiles, att, H, G, d, d ** -0.5, -small,
+                                         ctx.status, sink=sinks), flush=flush)
+            add(f"attention tcgen05, sinks, chunks of {small} {label}", us, T * (2 * H + 2 * G) * d * 2,
+                4 * n_seqs * (-(-q // small)) * (small * (small + 1) // 2) * H * d, like="attention tcgen05")
+        else:
+            keys = ctx_len + 1
+            splits = K.decode_splits(n_seqs, G, keys)
+            part_o, part_ml = torch.empty(n_seqs * H * splits * d, device=dev), torch.empty(n_seqs * H * splits * 2, device=dev)
+            kv_bytes = n_seqs * keys * 2 * G * d * 2 + T * 2 * H * d * 2
+            for name, sink, mask in (("attention decode, sinks, chunks", sinks, -MUMOPEL_CHUNK), ("attention decode", None, 0)):
+                us = _time(lambda: K.attn_decode(qkv, C, pages, table, ctx.cu_q, ctx_lens, n_seqs, att, part_o, part_ml, H, G, d,
+                                                 d ** -0.5, mask, splits, ctx.status, sink=sink), flush=flush)
+                add(f"{name} ({n_seqs} x {keys} keys)", us, kv_bytes, like="attention decode" if mask else None)
+        # -- the seam between two parts over the streams, beside the layer norm with the residual add
+        X = torch.randn(T, S, width, device=dev)
+        x0, y = torch.randn(T, width, device=dev), torch.randn(T, width, device=dev).to(bf)
+        mix, ow, iw = torch.eye(S, device=dev) * 0.9, torch.ones(S, device=dev), torch.full((S,), 1.0 / S, device=dev)
+        lw, lb, out = torch.ones(width, device=dev), torch.zeros(width, device=dev), torch.empty(T, width, dtype=bf, device=dev)
+        norm = dict(streams=S, in_w=iw, w=lw, b=lb, eps=1e-6)
+        us = _time(lambda: K.stream_seam(X, out, y=y, mix=mix, out_w=ow, dst=X, **norm), flush=flush)
+        add(f"seam over {S} streams {label} ({T} rows)", us, T * width * (8 * S + 2 + 2), like="layer norm with the residual add")
+        us = _time(lambda: K.stream_seam(x0, out, **norm), flush=flush)
+        add(f"seam at the model's start {label} ({T} rows)", us, T * width * (4 + 2), like="layer norm with the residual add")
+        n = T * TOP
+        outs, sh, wts = torch.randn(n, width, device=dev), torch.randn(T, width, device=dev), torch.rand(T, TOP, device=dev)
+        row_of = torch.randperm(n, device=dev).to(torch.int32)
+        us = _time(lambda: K.stream_seam(X, out, routed=(outs, row_of, wts, sh), mix=mix, out_w=ow, dst=X, **norm), flush=flush)
+        add(f"seam over {S} streams with the experts' sum {label} ({T} rows)", us, T * width * (8 * S + 4 * (TOP + 1) + 2),
+            like="experts' weighted sum")
+        us = _time(lambda: K.add_layer_norm(x0, y, lw, lb, 1e-6, out, None, 1.0), flush=flush)
+        add(f"layer norm with the residual add {label} ({T} rows)", us, T * width * (4 + 2 + 4 + 2))
+        us = _time(lambda: K.moe_combine(x0, outs, row_of, wts, sh, 1.0), flush=flush)
+        add(f"experts' weighted sum {label} ({T} rows)", us, T * width * 4 * (TOP + 3))
+        # -- the router's choice
+        z, bias = torch.randn(T, EXPERTS, device=dev), torch.randn(EXPERTS, device=dev)
+        ids = torch.empty(T, TOP, dtype=torch.int32, device=dev)
+        us = _time(lambda: K.moe_route(z, ids, wts, 1, 1, score=K.ROUTE_CHOSEN_SOFTMAX, renormalize=False, bias=bias), flush=flush)
+        add(f"route: softmax over the chosen, bias {label} ({T} rows)", us, T * (EXPERTS + 2 * TOP) * 4, like="route: softmax over all")
+        us = _time(lambda: K.moe_route(z, ids, wts, 1, 1), flush=flush)
+        add(f"route: softmax over all {label} ({T} rows)", us, T * (EXPERTS + 2 * TOP) * 4)
+        # -- the cap on the logits of a step's last tokens
+        lg = torch.randn(n_seqs, VOCAB, device=dev)
+        us = _time(lambda: K.softcap_(lg, 30.0), flush=flush)
+        add(f"cap on the logits ({n_seqs} rows)", us, lg.numel() * 8, like="logits times a constant")
+        us = _time(lambda: K.scale_(lg, 1.0), flush=flush)
+        add(f"logits times a constant ({n_seqs} rows)", us, lg.numel() * 8)
+        del pages, X, outs
+        torch.cuda.empty_cache()
+    return rows
+
+
+def mumopel_main(args, peaks: dict) -> int:
+    out = {"design": "Mumopel", "beside": "Qwen3 dense at equal width and layers, its feed-forward as wide as the experts a token uses plus the "
+                                          f"shared one (Mumopel has {MUMOPEL_STREAMS} residual streams where Qwen3 has one)",
+           "dtype": args.dtype, "batch": args.batch, "prompt_len": args.prompt_len, "new_tokens": args.steps,
+           "data": "synthetic token ids, seeded random weights", "peaks": peaks.get("source"), "sizes": {}}
+    for name, size in SIZES.items():
+        if args.design_sizes and name not in args.design_sizes.split(","):
+            continue
+        ours = run_engine(mumopel_config(**size), args.dtype, args.batch, args.prompt_len, args.steps)
+        beside = run_engine(qwen3_config(**size, max_len=args.prompt_len + args.steps + 64), args.dtype, args.batch, args.prompt_len, args.steps)
+        out["sizes"][name] = {"shape": size, "mumopel": ours, "qwen3": beside,
+                              "kernels": mumopel_kernel_table(size["width"], size["ff"], args.batch, args.prompt_len, peaks)}
         print(json.dumps({"partial": name, **out["sizes"][name]}), flush=True)
     print(json.dumps(out))
     return 0
