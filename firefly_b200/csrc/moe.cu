@@ -15,20 +15,12 @@
 //
 // A row of a grouped product is one (token, choice) pair; its result is a plain dot product
 // per output in a fixed order over K, so it does not depend on which other rows share its tile.
-#include "common.cuh"
+#include "moe.cuh"
 #include <math_constants.h>
 
 namespace ff {
 
 constexpr int MOE_BM = 64, MOE_BN = 64, MOE_BK = 16;
-
-// act 1: silu(g) * u, no clamps.  act 0: the clamped form below.
-__device__ __forceinline__ float clamped_glu(float g, float u, float limit, int act = 0) {
-    if (act == 1) return g / (1.0f + expf(-g)) * u;
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
-}
 
 // (value, index) arg-max over a warp; the lowest index wins ties
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
@@ -174,9 +166,6 @@ __global__ void moe_plan_kernel(const int* ids, const float* wts, float* __restr
 // out[row, n] = clamped_glu(gate, up) in type T.  MOE_UP: one B matrix, gathered rows, out = relu(up)^2 in type T.
 // MOE_DOWN: A = rows of `a` in place, out 32-bit.  `row_w` (or null; not MOE_DOWN): a row's products are multiplied by
 // row_w[row] in front of the activation, which is a weight on the expert's input.
-enum { MOE_DOWN = 0, MOE_GATEUP = 1, MOE_UP = 2 };
-__device__ __forceinline__ float relu2(float z) { z = fmaxf(z, 0.f); return z * z; }
-
 template <typename T, int KIND>
 __global__ void __launch_bounds__(256) moe_grouped_kernel(
     const T* a, const int* src_tok, const T* __restrict__ b0, const T* __restrict__ b1,

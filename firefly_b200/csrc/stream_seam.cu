@@ -36,6 +36,7 @@ struct SeamArgs {
     void* out;
     const int* row_idx;
     int W, kind, top, same, out_bf16;
+    int n_in;                  // numbers in in_w
 };
 
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -81,7 +82,9 @@ __global__ void __launch_bounds__(1024) stream_seam_vec_kernel(SeamArgs A) {
         float c = 0.f;
         if (i < S * S) c = A.kind != Y_NONE ? A.mix[i] : 0.f;
         else if (i < S * S + S) c = A.kind != Y_NONE ? A.out_w[i - S * S] : 0.f;
-        else c = A.in_w ? A.in_w[i - S * S - S] : 1.0f;
+        else if (S == 1 && A.n_in > 1) {                      // equal streams read at once: one row times the sum of the weights
+            for (int q = 0; q < A.n_in; ++q) c += A.in_w ? A.in_w[q] : 1.0f;
+        } else c = A.in_w ? A.in_w[i - S * S - S] : 1.0f;
         s_c[i] = c;
     }
     const float* mix = s_c;
@@ -243,11 +246,11 @@ FF_EXPORT int ff_stream_seam(const float* src, float* dst, const void* y, int y_
     if ((y_kind == Y_FLOAT || y_kind == Y_BF16) && !y) return FF_ERR_BAD_ARG;
     if (y_kind == Y_ROUTED && (!rows || !row_of || !wts || top <= 0)) return FF_ERR_BAD_ARG;
     if (dst && (row_idx || y_kind == Y_NONE || (same && dst == src))) return FF_ERR_BAD_ARG;
-    SeamArgs A{src, dst, y, rows, row_of, wts, shared, mix, out_w, in_w, w, b, eps, center, out, row_idx, W, y_kind, top, same, out_dtype};
+    SeamArgs A{src, dst, y, rows, row_of, wts, shared, mix, out_w, in_w, w, b, eps, center, out, row_idx, W, y_kind, top, same, out_dtype, S};
     const bool aligned = (((uintptr_t)src | (uintptr_t)dst | (uintptr_t)y | (uintptr_t)rows | (uintptr_t)shared | (uintptr_t)w |
                            (uintptr_t)b | (uintptr_t)out) & 15) == 0;
     if (aligned && W % 4 == 0 && W <= 16384 && S <= SEAM_FIXED_STREAMS) {
-        switch (S) {
+        switch (same && y_kind == Y_NONE ? 1 : S) {
             case 1: return seam_vec<1>(A, rows_out, stream);
             case 2: return seam_vec<2>(A, rows_out, stream);
             case 3: return seam_vec<3>(A, rows_out, stream);

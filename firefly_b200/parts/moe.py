@@ -178,11 +178,11 @@ class GroupedExperts(Part):
         plan = (seg, tile_e, tile_r, n_tiles, max_tiles)
         act = ws.get("moe.act", (rows, self.ff), dt)
         if self.gated:
-            K.moe_grouped(x, src_tok, self.w_gate, self.w_up, plan, act, self.limit, tc, self.activation, row_w=row_w)
+            K.moe_grouped(x, src_tok, self.w_gate, self.w_up, plan, act, self.limit, tc, self.activation, row_w=row_w, status=ctx.status)
         else:
-            K.moe_grouped(x, src_tok, self.w_up, None, plan, act, 0.0, tc, kind=K.MOE_UP, row_w=row_w)
+            K.moe_grouped(x, src_tok, self.w_up, None, plan, act, 0.0, tc, kind=K.MOE_UP, row_w=row_w, status=ctx.status)
         outs = ws.get("moe.rows", (rows, W), torch.float32)
-        K.moe_grouped(act, src_tok, self.w_down, None, plan, outs, 0.0, tc)
+        K.moe_grouped(act, src_tok, self.w_down, None, plan, outs, 0.0, tc, status=ctx.status)
         shared = None
         if self.shared_ff:
             sact = ws.get("moe.sh_act", (T, self.shared_ff), dt)
