@@ -117,48 +117,96 @@ __global__ void moe_route_kernel(const float* z, int z_stride, const float* __re
     }
 }
 
-// One block: rows sorted by expert.  seg[e] .. seg[e+1] are expert e's rows; row_of[entry] is
-// the row of (token, choice) = entry; src_tok[row] its token; the row tiles of row_tile rows
-// (64 for the plain grouped kernel, 128 for the tensor-core one) are listed as (expert, first row) with their count in n_tiles.
+// Rows sorted by expert, by one block or by a cluster of them (each takes a run of the entries; they share their counts
+// through distributed shared memory).  seg[e] .. seg[e+1] are expert e's rows; row_of[entry] is the row of
+// (token, choice) = entry; src_tok[row] its token; the row tiles of row_tile rows (64 for the plain grouped kernel, 128 for
+// the tensor-core one) are listed as (expert, first row) with their count in n_tiles.
 // `wts` (or null): row_w[row] becomes the weight of the row's (token, choice).
-__global__ void moe_plan_kernel(const int* ids, const float* wts, float* __restrict__ row_w, int entries, int top, int E, int row_tile, int* __restrict__ seg,
-                                int* __restrict__ row_of, int* __restrict__ src_tok, int* __restrict__ tile_expert,
-                                int* __restrict__ tile_row0, int* __restrict__ n_tiles) {
+constexpr int PLAN_THREADS = 1024, PLAN_BLOCKS = 8, PLAN_U = 8;
+__global__ void __launch_bounds__(PLAN_THREADS)
+moe_plan_kernel(const int* ids, const float* wts, float* __restrict__ row_w, int entries, int top, int E, int row_tile, int* __restrict__ seg,
+                int* __restrict__ row_of, int* __restrict__ src_tok, int* __restrict__ tile_expert, int* __restrict__ tile_row0,
+                int* __restrict__ n_tiles) {
     pdl_prologue();
     ids = pdl_fresh(ids);
     wts = pdl_fresh(wts);
     extern __shared__ int shi[];
-    int* counts = shi;
-    int* offs = shi + E;
-    int* cursor = offs + E + 1;
-    for (int e = threadIdx.x; e < E; e += blockDim.x) { counts[e] = 0; cursor[e] = 0; }
+    int* counts = shi;                // of this block's entries
+    int* total = shi + E;
+    int* cursor = total + E;          // next free row of an expert for this block
+    const int rank = blockIdx.z, blocks = gridDim.z, tid = threadIdx.x;
+    const int per = (entries + blocks - 1) / blocks, lo = min(entries, rank * per), hi = min(entries, lo + per);
+    for (int e = tid; e < E; e += PLAN_THREADS) counts[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < entries; i += blockDim.x) atomicAdd(&counts[ids[i]], 1);
+    for (int i0 = lo + tid; i0 < hi; i0 += PLAN_THREADS * PLAN_U) {       // several entries' loads in flight at once
+        int e[PLAN_U];
+#pragma unroll
+        for (int u = 0; u < PLAN_U; ++u) e[u] = i0 + u * PLAN_THREADS < hi ? ids[i0 + u * PLAN_THREADS] : -1;
+#pragma unroll
+        for (int u = 0; u < PLAN_U; ++u)
+            if (e[u] >= 0) atomicAdd(&counts[e[u]], 1);
+    }
     __syncthreads();
-    if (threadIdx.x == 0) {
-        int run = 0, nt = 0;
-        for (int e = 0; e < E; ++e) {
-            offs[e] = run;
-            seg[e] = run;
-            for (int r0 = 0; r0 < counts[e]; r0 += row_tile) {
-                tile_expert[nt] = e;
-                tile_row0[nt] = run + r0;
-                ++nt;
+    if (blocks > 1) cluster_sync_all();
+    for (int e = tid; e < E; e += PLAN_THREADS) {
+        int all = 0, before = 0;
+        if (blocks > 1) {
+            const uint32_t addr = (uint32_t)__cvta_generic_to_shared(counts + e);
+            for (int r = 0; r < blocks; ++r) {
+                const int c = __float_as_int(ld_peer_smem(addr, (uint32_t)r));
+                if (r < rank) before += c;
+                all += c;
             }
-            run += counts[e];
+        } else {
+            all = counts[e];
         }
-        offs[E] = run;
-        seg[E] = run;
-        n_tiles[0] = nt;
+        total[e] = all;
+        cursor[e] = before;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < entries; i += blockDim.x) {
-        const int e = ids[i];
-        const int row = offs[e] + atomicAdd(&cursor[e], 1);
-        row_of[i] = row;
-        src_tok[row] = i / top;
-        if (wts) row_w[row] = wts[i];
+    if (tid < 32) {                   // running sums over the experts: rows and row tiles
+        int rows0 = 0, tiles0 = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + tid, c = e < E ? total[e] : 0, nt = (c + row_tile - 1) / row_tile;
+            int rs = c, ts = nt;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int a = __shfl_up_sync(0xffffffffu, rs, o), b = __shfl_up_sync(0xffffffffu, ts, o);
+                if (tid >= o) { rs += a; ts += b; }
+            }
+            const int first = rows0 + rs - c;
+            if (e < E) {
+                cursor[e] += first;
+                if (rank == 0) {
+                    seg[e] = first;
+                    for (int k = 0, at = tiles0 + ts - nt; k < nt; ++k) { tile_expert[at + k] = e; tile_row0[at + k] = first + k * row_tile; }
+                }
+            }
+            rows0 += __shfl_sync(0xffffffffu, rs, 31);
+            tiles0 += __shfl_sync(0xffffffffu, ts, 31);
+        }
+        if (rank == 0 && tid == 0) { seg[E] = rows0; n_tiles[0] = tiles0; }
     }
+    __syncthreads();
+    for (int i0 = lo + tid; i0 < hi; i0 += PLAN_THREADS * PLAN_U) {
+        int e[PLAN_U];
+        float w[PLAN_U];
+#pragma unroll
+        for (int u = 0; u < PLAN_U; ++u) {
+            const int i = i0 + u * PLAN_THREADS;
+            e[u] = i < hi ? ids[i] : -1;
+            w[u] = wts && i < hi ? wts[i] : 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < PLAN_U; ++u) {
+            if (e[u] < 0) continue;
+            const int i = i0 + u * PLAN_THREADS, row = atomicAdd(&cursor[e[u]], 1);
+            row_of[i] = row;
+            src_tok[row] = i / top;
+            if (wts) row_w[row] = w[u];
+        }
+    }
+    if (blocks > 1) cluster_sync_all();      // a peer may still be reading this block's counts
 }
 
 // out rows = A rows x B[e]^T for the row tile's expert e.  B: [E, N, K] row-major.
@@ -235,148 +283,6 @@ __global__ void __launch_bounds__(256) moe_grouped_kernel(
     }
 }
 
-// The same grouped product for bfloat16 on tensor cores: mma.sync m16n8k16 with 32-bit accumulation,
-// operands staged through a three-stage cp.async ring in shared memory (rows padded to 40 elements so
-// that the 32-bit fragment loads of a warp fall into 32 different banks).  A block takes 128 rows of one
-// expert (the plan is made with that row tile) and 128 rows of B: 64 columns of gate and the same 64 of up
-// when GATEUP, else 128 output columns.  Eight warps in a 2 x 4 grid, each 64 rows x 32 rows of B (16 gate +
-// 16 up columns, so that a thread holds both halves of an output).  Needs K % 8 == 0 (16-byte copies).  Rows
-// past the expert's last row and columns past N are filled with zeros by the copies and not stored.
-constexpr int MMA_BM = 128, MMA_BR = 128, MMA_BK = 32, MMA_LD = 40, MMA_STAGES = 3;
-constexpr size_t MMA_SMEM = (size_t)MMA_STAGES * (MMA_BM + MMA_BR) * MMA_LD * sizeof(bf16);
-
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool pred) {
-    const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem);
-    const int bytes = pred ? 16 : 0;
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void mma_bf16_16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-template <int KIND>
-__global__ void __launch_bounds__(256) moe_grouped_mma_kernel(
-    const bf16* a, const int* src_tok, const bf16* __restrict__ b0,
-    const bf16* __restrict__ b1, const int* seg, const int* tile_expert,
-    const int* tile_row0, const int* n_tiles, const float* row_w, void* __restrict__ out, int N, int K,
-    float limit, int act) {
-    constexpr bool GATEUP = KIND == MOE_GATEUP, GATHER = KIND != MOE_DOWN;
-    pdl_prologue();
-    a = pdl_fresh(a); src_tok = pdl_fresh(src_tok); seg = pdl_fresh(seg);       // made by the kernels in front
-    row_w = pdl_fresh(row_w);
-    tile_expert = pdl_fresh(tile_expert); tile_row0 = pdl_fresh(tile_row0); n_tiles = pdl_fresh(n_tiles);
-    if ((int)blockIdx.y >= n_tiles[0]) return;
-    extern __shared__ __align__(16) unsigned char mma_smem[];
-    typedef bf16 (*Tile)[MMA_BM][MMA_LD];                      // [stage][row][k]
-    Tile As = reinterpret_cast<Tile>(mma_smem);
-    Tile Bs = reinterpret_cast<Tile>(mma_smem + (size_t)MMA_STAGES * MMA_BM * MMA_LD * sizeof(bf16));
-    static_assert(MMA_BM == MMA_BR, "A and B tiles share a shape");
-    constexpr int COLS = GATEUP ? MMA_BR / 2 : MMA_BR;          // output columns of a block
-    const int e = tile_expert[blockIdx.y], row0 = tile_row0[blockIdx.y];
-    const int rows = min(MMA_BM, seg[e + 1] - row0);
-    const int n0 = blockIdx.x * COLS;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int wm = warp >> 2, wn = warp & 3, g = lane >> 2, t4 = lane & 3;
-    // this thread's copies: rows tid / 4 and tid / 4 + 64 (of A and of B), 16-byte chunk tid % 4 of a stage's 32 columns.
-    // Row r of the B tile: GATEUP: warp wn's 32 rows are gate columns [16 wn, 16 wn + 16) then the same up columns;
-    // else output column r.
-    const int lr = tid >> 2, lc = (tid & 3) * 8;
-    const bf16* a_row[2];
-    const bf16* b_row[2];
-    bool a_ok[2], b_ok[2];
-#pragma unroll
-    for (int q = 0; q < 2; ++q) {
-        const int r = lr + 64 * q;
-        a_ok[q] = r < rows;
-        const int src = a_ok[q] ? (GATHER ? src_tok[row0 + r] : row0 + r) : 0;
-        a_row[q] = a + (size_t)src * K;
-        int col;
-        const bf16* base = b0;
-        if (GATEUP) {
-            const int w = r >> 5, in = r & 31;
-            col = n0 + w * 16 + (in & 15);
-            if (in >= 16) base = b1;
-        } else {
-            col = n0 + r;
-        }
-        b_ok[q] = col < N;
-        b_row[q] = base + ((size_t)e * N + (b_ok[q] ? col : 0)) * K;
-    }
-    const int KT = (K + MMA_BK - 1) / MMA_BK;
-    auto load = [&](int stage, int kt) {
-        const int k = kt * MMA_BK + lc;
-        const bool in = k < K;
-#pragma unroll
-        for (int q = 0; q < 2; ++q) {
-            cp_async16(&As[stage][lr + 64 * q][lc], a_row[q] + (in ? k : 0), in && a_ok[q]);
-            cp_async16(&Bs[stage][lr + 64 * q][lc], b_row[q] + (in ? k : 0), in && b_ok[q]);
-        }
-    };
-    float acc[4][4][4] = {};
-    for (int s = 0; s < MMA_STAGES - 1; ++s) {
-        if (s < KT) load(s, s);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    }
-    for (int kt = 0; kt < KT; ++kt) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(MMA_STAGES - 2) : "memory");
-        __syncthreads();
-        const int nxt = kt + MMA_STAGES - 1;
-        if (nxt < KT) load(nxt % MMA_STAGES, nxt);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        const int st = kt % MMA_STAGES;
-#pragma unroll
-        for (int kk = 0; kk < MMA_BK; kk += 16) {
-            uint32_t bfr[4][2];
-#pragma unroll
-            for (int nt = 0; nt < 4; ++nt) {
-                const int n = wn * 32 + nt * 8 + g;
-                bfr[nt][0] = *reinterpret_cast<const uint32_t*>(&Bs[st][n][kk + 2 * t4]);
-                bfr[nt][1] = *reinterpret_cast<const uint32_t*>(&Bs[st][n][kk + 8 + 2 * t4]);
-            }
-#pragma unroll
-            for (int mt = 0; mt < 4; ++mt) {
-                const int r = wm * 64 + mt * 16 + g;
-                uint32_t af[4];
-                af[0] = *reinterpret_cast<const uint32_t*>(&As[st][r][kk + 2 * t4]);
-                af[1] = *reinterpret_cast<const uint32_t*>(&As[st][r + 8][kk + 2 * t4]);
-                af[2] = *reinterpret_cast<const uint32_t*>(&As[st][r][kk + 8 + 2 * t4]);
-                af[3] = *reinterpret_cast<const uint32_t*>(&As[st][r + 8][kk + 8 + 2 * t4]);
-#pragma unroll
-                for (int nt = 0; nt < 4; ++nt) mma_bf16_16816(acc[mt][nt], af, bfr[nt][0], bfr[nt][1]);
-            }
-        }
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-#pragma unroll
-    for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            const int r = wm * 64 + mt * 16 + g + (c >> 1) * 8;
-            if (r >= rows) continue;
-            const float wr = GATHER && row_w ? row_w[row0 + r] : 1.0f;
-            if (GATEUP) {
-                // B rows 0..15 of the warp are gate (n tiles 0, 1), rows 16..31 the same columns of up (n tiles 2, 3)
-#pragma unroll
-                for (int nt = 0; nt < 2; ++nt) {
-                    const int n = n0 + wn * 16 + nt * 8 + 2 * t4 + (c & 1);
-                    if (n < N)
-                        ((bf16*)out)[(size_t)(row0 + r) * N + n] =
-                            __float2bfloat16_rn(clamped_glu(acc[mt][nt][c] * wr, acc[mt][nt + 2][c] * wr, limit, act));
-                }
-            } else {
-#pragma unroll
-                for (int nt = 0; nt < 4; ++nt) {
-                    const int n = n0 + wn * 32 + nt * 8 + 2 * t4 + (c & 1);
-                    if (n >= N) continue;
-                    if (KIND == MOE_UP) ((bf16*)out)[(size_t)(row0 + r) * N + n] = __float2bfloat16_rn(relu2(acc[mt][nt][c] * wr));
-                    else ((float*)out)[(size_t)(row0 + r) * N + n] = acc[mt][nt][c];
-                }
-            }
-        }
-}
-
 // y[t, f] = clamped_glu(gu[t, f], gu[t, F + f])
 template <typename T>
 __global__ void clamped_glu_kernel(const T* gu, T* __restrict__ y, int F, float limit, size_t total) {
@@ -414,7 +320,7 @@ __global__ void moe_combine_kernel(float* __restrict__ residual, const float* ro
 using namespace ff;
 
 // rows of a row tile: of the tensor-core kernel (bfloat16, K % 8 == 0) or of the plain one
-FF_EXPORT int ff_moe_row_tile(int tensor_cores) { return tensor_cores ? MMA_BM : MOE_BM; }
+FF_EXPORT int ff_moe_row_tile(int tensor_cores) { return tensor_cores ? GROUPED_TC_ROWS : MOE_BM; }
 
 FF_EXPORT int ff_moe_route(const float* z, int z_stride, const float* bias, const float* correction, int T, int E, int top, int groups, int keep,
                            int score, int group_score, int renorm, int* ids, float* wts, cudaStream_t stream) {
@@ -434,39 +340,23 @@ FF_EXPORT int ff_moe_route(const float* z, int z_stride, const float* bias, cons
 FF_EXPORT int ff_moe_plan(const int* ids, const float* wts, float* row_w, int entries, int top, int E, int row_tile, int* seg, int* row_of,
                           int* src_tok, int* tile_expert, int* tile_row0, int* n_tiles, cudaStream_t stream) {
     if (entries <= 0) return 0;
-    if ((row_tile != MOE_BM && row_tile != MMA_BM) || (wts && !row_w)) return FF_ERR_BAD_ARG;
-    const size_t smem = (size_t)(3 * E + 1) * sizeof(int);
+    if ((row_tile != MOE_BM && row_tile != GROUPED_TC_ROWS) || (wts && !row_w)) return FF_ERR_BAD_ARG;
+    const size_t smem = (size_t)3 * E * sizeof(int);
     if (smem > 48 * 1024) return FF_ERR_UNSUPPORTED;
-    FF_LAUNCH(moe_plan_kernel, 1, 1024, smem, stream, ids, wts, row_w, entries, top, E, row_tile, seg, row_of, src_tok, tile_expert,
-              tile_row0, n_tiles);
+    const int blocks = entries >= 4096 ? PLAN_BLOCKS : 1;
+    const int rc = launch_kernel_cluster(moe_plan_kernel, dim3(1, 1, blocks), dim3(PLAN_THREADS), smem, stream, blocks, ids, wts, row_w,
+                                         entries, top, E, row_tile, seg, row_of, src_tok, tile_expert, tile_row0, n_tiles);
+    if (rc) return rc;
     FF_LAUNCH_CHECK();
     return 0;
 }
 
 FF_EXPORT int ff_moe_grouped(const void* a, const int* src_tok, const void* b0, const void* b1, int dtype, int kind,
                              const int* seg, const int* tile_expert, const int* tile_row0, const int* n_tiles,
-                             const float* row_w, void* out, int max_tiles, int N, int K, float limit, int act, int tensor_cores,
+                             const float* row_w, void* out, int max_tiles, int N, int K, float limit, int act,
                              cudaStream_t stream) {
     if (max_tiles <= 0) return 0;
     if (kind < MOE_DOWN || kind > MOE_UP || (kind == MOE_GATEUP && !b1)) return FF_ERR_BAD_ARG;
-    if (tensor_cores) {
-        // the plan was made with 128-row tiles
-        if (dtype != 1 || K % 8 || ((((uintptr_t)a | (uintptr_t)b0 | (uintptr_t)b1) & 15) != 0)) return FF_ERR_BAD_ARG;
-        const int cols = kind == MOE_GATEUP ? MMA_BR / 2 : MMA_BR;
-        dim3 grid((N + cols - 1) / cols, max_tiles);
-#define FF_MOE_TC(KIND)                                                                                             \
-    do {                                                                                                            \
-        FF_SMEM_LIMIT((moe_grouped_mma_kernel<KIND>), MMA_SMEM);                                                    \
-        FF_LAUNCH((moe_grouped_mma_kernel<KIND>), grid, 256, MMA_SMEM, stream, (const bf16*)a, src_tok, (const bf16*)b0, \
-                  (const bf16*)b1, seg, tile_expert, tile_row0, n_tiles, row_w, out, N, K, limit, act);             \
-    } while (0)
-        if (kind == MOE_GATEUP) FF_MOE_TC(MOE_GATEUP);
-        else if (kind == MOE_UP) FF_MOE_TC(MOE_UP);
-        else FF_MOE_TC(MOE_DOWN);
-#undef FF_MOE_TC
-        FF_LAUNCH_CHECK();
-        return 0;
-    }
     dim3 grid((N + MOE_BN - 1) / MOE_BN, max_tiles);
 #define FF_MOE(T, KIND)                                                                                            \
     FF_LAUNCH((moe_grouped_kernel<T, KIND>), grid, 256, 0, stream, (const T*)a, src_tok, (const T*)b0, (const T*)b1, seg, \

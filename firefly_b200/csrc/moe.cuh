@@ -24,6 +24,8 @@ __device__ __forceinline__ float clamped_glu_fast(float g, float u, float limit,
     return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
 }
 
+constexpr int GROUPED_TC_ROWS = 128;      // rows of a row tile of the tensor-core product
+
 __device__ __forceinline__ float relu2(float z) { z = fmaxf(z, 0.f); return z * z; }
 
 }  // namespace ff

@@ -16,7 +16,7 @@
 
 namespace ff {
 
-constexpr int GM = 128;               // rows of a row tile (MMA M)
+constexpr int GM = GROUPED_TC_ROWS;   // rows of a row tile (MMA M)
 constexpr int GROUPED_THREADS = 192;  // a warp for the loads, one for the MMAs, four for the epilogue
 
 template <int BC> struct GroupedCfg {

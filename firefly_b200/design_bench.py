@@ -175,9 +175,10 @@ def kernel_table(width: int, ff: int, batch: int, prompt: int, peaks: dict) -> l
         wd = torch.randn(E, width, ff, device=dev).to(bf) * 0.02
         act, outs = torch.empty(n, ff, dtype=bf, device=dev), torch.empty(n, width, device=dev)
         used = min(E, n)
-        us = _time(lambda: K.moe_grouped(xa, ints[2], wg, wu, plan, act, 7.0, True), flush=flush)
+        status = torch.zeros(1, dtype=torch.int32, device=dev)
+        us = _time(lambda: K.moe_grouped(xa, ints[2], wg, wu, plan, act, 7.0, True, status=status), flush=flush)
         add(f"moe gate|up {label} ({n} rows)", us, bytes_=used * 2 * ff * width * 2 + n * (width + ff) * 2, flops=4 * n * ff * width)
-        us = _time(lambda: K.moe_grouped(act, ints[2], wd, None, plan, outs, 0.0, True), flush=flush)
+        us = _time(lambda: K.moe_grouped(act, ints[2], wd, None, plan, outs, 0.0, True, status=status), flush=flush)
         add(f"moe down {label} ({n} rows)", us, bytes_=used * ff * width * 2 + n * (ff * 2 + width * 4), flops=2 * n * ff * width)
         # the dense model's like kernel: its gate|up product at the same number of operations
         inter = top * ff
@@ -848,10 +849,10 @@ def gatutar_kernel_table(width: int, ff: int, batch: int, prompt: int, peaks: di
         up, gate = ((torch.randn(E, F, width, device=dev) * 0.02).to(bf) for _ in range(2))
         act = torch.empty(n, F, dtype=bf, device=dev)
         used = min(E, n)
-        us = _time(lambda: K.moe_grouped(x, src, up, None, plan, act, 0.0, True, kind=K.MOE_UP, row_w=row_w), flush=flush)
+        us = _time(lambda: K.moe_grouped(x, src, up, None, plan, act, 0.0, True, kind=K.MOE_UP, row_w=row_w, status=ctx.status), flush=flush)
         add(f"experts' first product, ungated, weighted {label} ({n} rows)", us, used * F * width * 2 + T * width * 2 + n * F * 2,
             2 * n * F * width, like="experts' first product, gated")
-        us = _time(lambda: K.moe_grouped(x, src, gate, up, plan, act, 0.0, True, K.GLU_SILU), flush=flush)
+        us = _time(lambda: K.moe_grouped(x, src, gate, up, plan, act, 0.0, True, K.GLU_SILU, status=ctx.status), flush=flush)
         add(f"experts' first product, gated {label} ({n} rows)", us, 2 * used * F * width * 2 + T * width * 2 + n * F * 2, 4 * n * F * width)
         outs, sh, z = torch.randn(n, width, device=dev), torch.randn(T, width, device=dev), torch.randn(T, E + 1, device=dev)
         us = _time(lambda: K.moe_combine(res, outs, row_of, None, sh, 1.0, top=TOP, shared_z=z[:, E], overwrite=True), flush=flush)
@@ -909,6 +910,7 @@ def mumopel_kernel_table(width: int, ff: int, batch: int, prompt: int, peaks: di
     """The kernels that Mumopel added or changed, alone against their floors, each beside the like kernel (or the same
     kernel without the new option) of the models that were there."""
     from .ops import kernels as K
+    from .parts.linear import linear_into_residual, linear_swiglu
     dev = torch.device("cuda:0")
     bf = torch.bfloat16
     flush = torch.empty(192 << 20, dtype=torch.uint8, device=dev)
@@ -993,6 +995,34 @@ def mumopel_kernel_table(width: int, ff: int, batch: int, prompt: int, peaks: di
         add(f"route: softmax over the chosen, bias {label} ({T} rows)", us, T * (EXPERTS + 2 * TOP) * 4, like="route: softmax over all")
         us = _time(lambda: K.moe_route(z, ids, wts, 1, 1), flush=flush)
         add(f"route: softmax over all {label} ({T} rows)", us, T * (EXPERTS + 2 * TOP) * 4)
+        # -- the experts' plan and grouped products, beside the dense feed-forward's products of as many operations
+        E = EXPERTS
+        x = (torch.randn(T, width, device=dev) * 0.5).to(bf)
+        tiles = K.moe_max_tiles(n, E, True)
+        i32 = dict(dtype=torch.int32, device=dev)
+        seg, row_p, src, te, tr, nt = (torch.empty(k, **i32) for k in (E + 1, n, n, tiles, tiles, 1))
+        us = _time(lambda: K.moe_plan(ids, E, seg, row_p, src, te, tr, nt, True), flush=flush)
+        add(f"experts' plan {label} ({n} rows)", us, n * (4 + 4 + 4))
+        plan = (seg, te, tr, nt, tiles)
+        up, gate = ((torch.randn(E, ff, width, device=dev) * 0.02).to(bf) for _ in range(2))
+        down = (torch.randn(E, width, ff, device=dev) * 0.02).to(bf)
+        act = torch.empty(n, ff, dtype=bf, device=dev)
+        used = min(E, n)
+        us = _time(lambda: K.moe_grouped(x, src, gate, up, plan, act, 7.0, True, status=ctx.status), flush=flush)
+        add(f"experts' first product and activation {label} ({n} rows)", us, 2 * used * ff * width * 2 + T * width * 2 + n * ff * 2,
+            4 * n * ff * width, like="dense gate|up product and SwiGLU")
+        us = _time(lambda: K.moe_grouped(act, src, down, None, plan, outs, 0.0, True, status=ctx.status), flush=flush)
+        add(f"experts' second product {label} ({n} rows)", us, used * ff * width * 2 + n * ff * 2 + n * width * 4, 2 * n * ff * width,
+            like="dense down product")
+        inter = TOP * ff
+        wgu = (torch.randn(2 * inter, width, device=dev) * 0.02).to(bf)
+        wdn = (torch.randn(width, inter, device=dev) * 0.02).to(bf)
+        da = torch.zeros(T, inter, dtype=bf, device=dev)
+        step = SimpleNamespace(workspace=_Scratch(dev), dtype=bf, status=ctx.status)
+        us = _time(lambda: linear_swiglu(x, wgu, inter, True, step), flush=flush)
+        add(f"dense gate|up product and SwiGLU {label} ({T} rows of {inter})", us, 2 * inter * width * 2 + T * (width + inter) * 2, 4 * T * inter * width)
+        us = _time(lambda: linear_into_residual(da, wdn, x0, step, "down"), flush=flush)
+        add(f"dense down product {label} ({T} rows of {inter})", us, inter * width * 2 + T * inter * 2 + T * width * 8, 2 * T * inter * width)
         # -- the cap on the logits of a step's last tokens
         lg = torch.randn(n_seqs, VOCAB, device=dev)
         us = _time(lambda: K.softcap_(lg, 30.0), flush=flush)

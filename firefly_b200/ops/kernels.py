@@ -981,8 +981,7 @@ def latent_gate(val, g, y, heads: int, vdim: int, per_head: bool = False) -> Non
 
 # --------------------------------------------------------------------------- #
 # routed experts (csrc/moe.cu)
-USE_TCGEN05_MOE = True      # tests flip this to hold the tcgen05 grouped product against the mma.sync one
-MOE_WIDE_BLOCKS_PER_SM = 2  # the wide tiles (256 weight rows a block) as soon as they still fill the places
+MOE_WIDE_BLOCKS_PER_SM = 1.5   # tiles of 256 weight rows a block as soon as they come to this many blocks an SM, else of 128
 MOE_FORCE_PLAIN = False     # tests flip this to hold the tensor-core grouped product against the plain one
 
 
@@ -1053,8 +1052,7 @@ def moe_grouped(a, src_tok, b0, b1, plan, out, limit: float = 0.0, tensor_cores:
     or, with ``kind`` MOE_UP (experts without a gate), gathered rows and out[row] = relu(u)^2 in a's type.  ``row_w`` float32
     [rows] (first products): a row's products are multiplied by it in front of the activation.  ``plan`` = (seg, tile_expert, tile_row0, n_tiles,
     max_tiles), made with the same ``tensor_cores``: a tensor-core kernel (bfloat16, K % 8 == 0) or the plain one.
-    With ``status`` (int32 [1]: where a wait that runs out is told) the tensor-core kernel is the tcgen05 one, else the
-    mma.sync one."""
+    The tensor-core kernel (tcgen05) needs ``status`` (int32 [1]: where a wait that runs out is told)."""
     seg, tile_expert, tile_row0, n_tiles, max_tiles = plan
     _need_cuda(a, src_tok, b0, b1, out, row_w)
     if kind is None:
@@ -1064,7 +1062,10 @@ def moe_grouped(a, src_tok, b0, b1, plan, out, limit: float = 0.0, tensor_cores:
     assert a.shape[1] == Kd and a.dtype == b0.dtype and out.shape[1] == N
     assert out.dtype == (a.dtype if kind != MOE_DOWN else torch.float32)
     assert not tensor_cores or (a.dtype == torch.bfloat16 and Kd % 8 == 0)
-    if tensor_cores and status is not None and USE_TCGEN05_MOE:
+    if tensor_cores:
+        _need_cuda(status)
+        if status is None:
+            raise KernelError("moe_grouped: the tensor-core kernel needs a status word")
         cols = 128 if kind == MOE_GATE_UP else 256
         _check(_lib("moe_tcgen05").ff_moe_grouped_tc(
             _p(a), c_int(a.shape[0]), _p(src_tok), _p(b0), _p(b1), c_int(E), c_int(kind), _p(seg), _p(tile_expert), _p(tile_row0),
@@ -1073,8 +1074,7 @@ def moe_grouped(a, src_tok, b0, b1, plan, out, limit: float = 0.0, tensor_cores:
         return
     _check(_lib("moe").ff_moe_grouped(_p(a), _p(src_tok), _p(b0), _p(b1), c_int(_dt(a)), c_int(kind),
                                      _p(seg), _p(tile_expert), _p(tile_row0), _p(n_tiles), _p(row_w), _p(out), c_int(max_tiles),
-                                     c_int(N), c_int(Kd), c_float(limit), c_int(act),
-                                     c_int(1 if tensor_cores else 0), _stream()), "moe_grouped")
+                                     c_int(N), c_int(Kd), c_float(limit), c_int(act), _stream()), "moe_grouped")
 
 
 def clamped_glu(gu, y, limit: float) -> None:
