@@ -216,7 +216,10 @@ __global__ void stream_seam_kernel(SeamArgs A, int S) {
 template <int S>
 static int seam_vec(const SeamArgs& A, int rows, cudaStream_t stream) {
     const int groups = A.W / 4;
-    if (A.W <= 2048) {
+    if (rows <= 256 && A.W <= 4096) {                         // few rows: more threads a row, each with less to wait for
+        const int threads = ((groups + 31) / 32) * 32;
+        FF_LAUNCH((stream_seam_vec_kernel<S, 1>), rows, threads, 0, stream, A);
+    } else if (A.W <= 2048) {
         const int threads = (((groups + 1) / 2 + 31) / 32) * 32;
         FF_LAUNCH((stream_seam_vec_kernel<S, 2>), rows, threads, 0, stream, A);
     } else {

@@ -1023,6 +1023,12 @@ def mumopel_kernel_table(width: int, ff: int, batch: int, prompt: int, peaks: di
         add(f"dense gate|up product and SwiGLU {label} ({T} rows of {inter})", us, 2 * inter * width * 2 + T * (width + inter) * 2, 4 * T * inter * width)
         us = _time(lambda: linear_into_residual(da, wdn, x0, step, "down"), flush=flush)
         add(f"dense down product {label} ({T} rows of {inter})", us, inter * width * 2 + T * inter * 2 + T * width * 8, 2 * T * inter * width)
+        # -- the shared expert's activation, beside the dense one's
+        sgu, sy = (torch.randn(T, 4 * ff, device=dev)).to(bf), torch.empty(T, 2 * ff, dtype=bf, device=dev)
+        us = _time(lambda: K.clamped_glu(sgu, sy, 7.0), flush=flush)
+        add(f"shared expert's activation {label} ({T} rows of {2 * ff})", us, T * 2 * ff * 2 * 3, like="silu_mul")
+        us = _time(lambda: K.silu_mul(sgu, sy), flush=flush)
+        add(f"silu_mul {label} ({T} rows of {2 * ff})", us, T * 2 * ff * 2 * 3)
         # -- the cap on the logits of a step's last tokens
         lg = torch.randn(n_seqs, VOCAB, device=dev)
         us = _time(lambda: K.softcap_(lg, 30.0), flush=flush)

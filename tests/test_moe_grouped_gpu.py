@@ -130,3 +130,15 @@ def test_the_plan_sorts_every_choice_by_expert(T, E, top, tc):
     assert torch.equal(src[row_of.long()].long(), torch.arange(n) // top) and torch.equal(row_w[row_of.long()], wts.view(-1))
     want = [(k, int(seg[k]) + r) for k in range(E) for r in range(0, int(counts[k]), rt)]
     assert int(nt[0]) == len(want) <= tiles and list(zip(te.tolist(), tr.tolist()))[: len(want)] == want
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("T,F", [(1, 8), (3, 21), (64, 1024), (513, 40), (7, 36)])
+def test_the_clamped_activation(dtype, T, F):
+    from firefly_b200.ops import kernels as K
+    gu = (torch.randn(T, 2 * F, generator=torch.Generator().manual_seed(F)) * 2).to(dtype)
+    y = torch.empty(T, F, dtype=dtype, device="cuda")
+    K.clamped_glu(gu.cuda(), y, 1.25)
+    g, u = torch.clamp(gu[:, :F].double(), max=1.25), torch.clamp(gu[:, F:].double(), min=-1.25, max=1.25)
+    want = g * torch.sigmoid(1.702 * g) * (u + 1.0)
+    assert float((y.cpu().double() - want).abs().max()) <= (2e-6 if dtype == torch.float32 else 5e-3) * float(want.abs().max())
